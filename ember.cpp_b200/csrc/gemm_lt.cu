@@ -231,21 +231,21 @@ EMBER_API int ember_linear_bf16(const void* A, const void* W, const float* bias_
 // ---------------------------------------------------------------------------- one product per head
 // out[t, h * out_head + (0..N)] = a[t, h * a_head + (0..K)] . w[h]^T for every head h: the library's strided batch,
 // the heads side by side in the rows of `a` and `out` (a head's offset is the batch stride, a row's width the leading
-// dimension), w [heads, N, K].  bfloat16 in and out, float32 sums.  Returns 2 where the library offers no algorithm.
+// dimension), w [heads, N, K].  bfloat16 in, bfloat16 or float32 out, float32 sums.  Returns 2 where the library offers no algorithm.
 namespace {
 struct HeadKey {
   int T, N, K, heads;
   long long a_stride, out_stride;
-  int a_head, out_head, align;
+  int a_head, out_head, align, out_dtype;
   bool operator==(const HeadKey& o) const {
     return T == o.T && N == o.N && K == o.K && heads == o.heads && a_stride == o.a_stride && out_stride == o.out_stride &&
-           a_head == o.a_head && out_head == o.out_head && align == o.align;
+           a_head == o.a_head && out_head == o.out_head && align == o.align && out_dtype == o.out_dtype;
   }
 };
 struct HeadHash {
   size_t operator()(const HeadKey& k) const {
     size_t h = 1469598103934665603ull;
-    const long long v[9] = {k.T, k.N, k.K, k.heads, k.a_stride, k.out_stride, k.a_head, k.out_head, k.align};
+    const long long v[10] = {k.T, k.N, k.K, k.heads, k.a_stride, k.out_stride, k.a_head, k.out_head, k.align, k.out_dtype};
     for (long long x : v) h = (h ^ (size_t)x) * 1099511628211ull;
     return h;
   }
@@ -260,16 +260,18 @@ int lowest_bit_bytes(unsigned long long v) {   // the largest power of two up to
 }  // namespace
 
 EMBER_API int ember_head_linear_bf16(const void* a, long long a_stride, int a_head, const void* w, void* out,
-                                     long long out_stride, int out_head, int T, int heads, int N, int K, void* workspace,
-                                     size_t workspace_bytes, cudaStream_t stream) {
+                                     long long out_stride, int out_head, int T, int heads, int N, int K, int out_dtype,
+                                     void* workspace, size_t workspace_bytes, cudaStream_t stream) {
+  EMBER_CHECK(out_dtype == EMBER_BF16 || out_dtype == EMBER_F32, "head_linear_bf16: output type %d", out_dtype);
+  const unsigned long long ob = out_dtype == EMBER_F32 ? 4 : 2;
   EMBER_CHECK(T > 0 && heads > 0 && N > 0 && K > 0, "head_linear_bf16: bad sizes");
   // what every pointer of the batch is a multiple of: the bases, the rows and the heads' offsets
   int align = lowest_bit_bytes((unsigned long long)(uintptr_t)a | (unsigned long long)(uintptr_t)out |
                                (unsigned long long)(uintptr_t)w | (unsigned long long)a_stride * 2 |
-                               (unsigned long long)out_stride * 2 | (unsigned long long)a_head * 2 |
-                               (unsigned long long)out_head * 2 | (unsigned long long)K * 2 | (unsigned long long)N * K * 2);
+                               (unsigned long long)out_stride * ob | (unsigned long long)a_head * 2 |
+                               (unsigned long long)out_head * ob | (unsigned long long)K * 2 | (unsigned long long)N * K * 2);
   if (align < 16) return 2;
-  const HeadKey key{T, N, K, heads, a_stride, out_stride, a_head, out_head, align};
+  const HeadKey key{T, N, K, heads, a_stride, out_stride, a_head, out_head, align, out_dtype};
   std::lock_guard<std::mutex> lock(g_mutex);
   if (!g_handle) LT_TRY(cublasLtCreate(&g_handle));
   auto it = g_head_plans.find(key);
@@ -290,7 +292,7 @@ EMBER_API int ember_head_linear_bf16(const void* a, long long a_stride, int a_he
     LT_TRY(cublasLtMatmulDescSetAttribute(p.op, CUBLASLT_MATMUL_DESC_TRANSB, &tb, sizeof(tb)));
     LT_TRY(cublasLtMatrixLayoutCreate(&p.a, CUDA_R_16BF, K, N, K));                 // w[h] as K x N, ld K
     LT_TRY(cublasLtMatrixLayoutCreate(&p.b, CUDA_R_16BF, K, T, a_stride));          // a's head as K x T, ld a row
-    LT_TRY(cublasLtMatrixLayoutCreate(&p.c, CUDA_R_16BF, N, T, out_stride));        // out's head as N x T, ld a row
+    LT_TRY(cublasLtMatrixLayoutCreate(&p.c, out_dtype == EMBER_F32 ? CUDA_R_32F : CUDA_R_16BF, N, T, out_stride));  // out's head as N x T, ld a row
     const int32_t batch = heads;
     const int64_t sa = (int64_t)N * K, sb = a_head, sc = out_head;
     LT_TRY(cublasLtMatrixLayoutSetAttribute(p.a, CUBLASLT_MATRIX_LAYOUT_BATCH_COUNT, &batch, sizeof(batch)));

@@ -103,9 +103,9 @@ latent_rows_kernel(const float* __restrict__ down, int down_width, int q_rank, c
 
 // out[t, out_col + h * out_head + n] = sum_k a[t, a_col + h * a_head + k] * w[h][n][k], float32 sums in ascending k.
 // grid (ceil(T / 32), ceil(N / 32), heads), block (32, 8): a tile of 32 tokens x 32 outputs of one head.
-template <typename T>
+template <typename T, typename TO>
 __global__ void head_linear_kernel(const T* __restrict__ a, long long a_stride, int a_col, int a_head,
-                                   const T* __restrict__ w, T* __restrict__ out, long long out_stride, int out_col,
+                                   const T* __restrict__ w, TO* __restrict__ out, long long out_stride, int out_col,
                                    int out_head, int T_tokens, int N, int K) {
   __shared__ float as[32][33], ws[32][33];
   const int h = blockIdx.z, m0 = blockIdx.x * 32, n0 = blockIdx.y * 32;
@@ -132,7 +132,7 @@ __global__ void head_linear_kernel(const T* __restrict__ a, long long a_stride, 
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty + 8 * i, n = n0 + tx;
-    if (m < T_tokens && n < N) out[(size_t)m * out_stride + out_col + (size_t)h * out_head + n] = from_float<T>(acc[i]);
+    if (m < T_tokens && n < N) out[(size_t)m * out_stride + out_col + (size_t)h * out_head + n] = from_float<TO>(acc[i]);
   }
 }
 
@@ -279,19 +279,18 @@ EMBER_API int ember_latent_rows(const float* down, int down_width, int q_rank, c
 
 EMBER_API int ember_head_linear(const void* a, long long a_stride, int a_col, int a_head, const void* w, void* out,
                                 long long out_stride, int out_col, int out_head, int T, int heads, int N, int K, int dtype,
-                                cudaStream_t stream) {
+                                int out_dtype, cudaStream_t stream) {
   EMBER_CHECK(T > 0 && heads > 0 && heads <= 65535 && N > 0 && K > 0, "head_linear: bad sizes");
   EMBER_CHECK((N + 31) / 32 <= 65535, "head_linear: %d outputs exceed one launch", N);
   const dim3 grid((T + 31) / 32, (N + 31) / 32, heads), block(32, 8);
-  if (dtype == EMBER_F32)
-    head_linear_kernel<float><<<grid, block, 0, stream>>>((const float*)a, a_stride, a_col, a_head, (const float*)w,
-                                                          (float*)out, out_stride, out_col, out_head, T, N, K);
-  else if (dtype == EMBER_BF16)
-    head_linear_kernel<__nv_bfloat16><<<grid, block, 0, stream>>>((const __nv_bfloat16*)a, a_stride, a_col, a_head,
-                                                                  (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_stride,
-                                                                  out_col, out_head, T, N, K);
-  else
-    return ember_fail("head_linear: element type %d", dtype);
+#define EMBER_HL(T_, TO_)                                                                                                       \
+  head_linear_kernel<T_, TO_><<<grid, block, 0, stream>>>((const T_*)a, a_stride, a_col, a_head, (const T_*)w, (TO_*)out, out_stride, \
+                                                          out_col, out_head, T, N, K)
+  if (dtype == EMBER_F32 && out_dtype == EMBER_F32) EMBER_HL(float, float);
+  else if (dtype == EMBER_BF16 && out_dtype == EMBER_BF16) EMBER_HL(__nv_bfloat16, __nv_bfloat16);
+  else if (dtype == EMBER_BF16 && out_dtype == EMBER_F32) EMBER_HL(__nv_bfloat16, float);
+  else return ember_fail("head_linear: element types %d -> %d", dtype, out_dtype);
+#undef EMBER_HL
   EMBER_LAUNCH_OK("head_linear");
   return 0;
 }

@@ -324,7 +324,7 @@ __device__ __forceinline__ void warp_argmax(float& best, int& at) {
 
 __global__ void __launch_bounds__(32 * kPickWarps)
 moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int T, int experts, int top,
-                int groups, int keep, float scale, int* __restrict__ chosen, float* __restrict__ weights) {
+                int groups, int keep, float scale, int softmax, int* __restrict__ chosen, float* __restrict__ weights) {
   extern __shared__ float pick_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kPickWarps + warp;
@@ -333,9 +333,11 @@ moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restric
   float* ch = sc + experts;
   float* gs = ch + experts;
   for (int e = lane; e < experts; e += 32) {
-    const float s = 1.0f / (1.0f + expf(-logits[(size_t)t * ld + e]));
+    // (softmax: the stored vector is a bias of the logits, which are chosen by and weigh as they are)
+    const float z = logits[(size_t)t * ld + e];
+    const float s = softmax ? z + correction[e] : 1.0f / (1.0f + expf(-z));
     sc[e] = s;
-    ch[e] = s + correction[e];
+    ch[e] = softmax ? s : s + correction[e];
   }
   __syncwarp();
   if (groups > 1) {
@@ -372,7 +374,7 @@ moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restric
       if (gs[e / per] != INFINITY) ch[e] = -INFINITY;
     __syncwarp();
   }
-  float sum = 0.f;      // (every lane keeps the same sum)
+  float sum = 0.f, first = 0.f;      // (every lane keeps the same sum, and the first choice's logit)
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
@@ -385,10 +387,12 @@ moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restric
     }
     warp_argmax(best, at);
     if (at >= experts) at = 0;
-    sum += sc[at];
+    if (softmax && k == 0) first = sc[at];      // (within one group of experts the largest comes first)
+    const float wt = softmax ? expf(sc[at] - first) : sc[at];
+    sum += wt;
     if (lane == 0) {
       chosen[(size_t)t * top + k] = at;
-      weights[(size_t)t * top + k] = sc[at];
+      weights[(size_t)t * top + k] = wt;
       ch[at] = -INFINITY;
     }
     __syncwarp();
@@ -416,16 +420,18 @@ moe_combine_kernel(const float* __restrict__ x, const float* __restrict__ y, con
 }  // namespace
 
 // logits float32 [T, ld] (the first `experts` columns are the router's), correction float32 [experts];
-// chosen int32 [T, top], weights float32 [T, top].
+// chosen int32 [T, top], weights float32 [T, top].  softmax 0: scores sigmoid(z), chosen by score + correction, weights the
+// chosen's scores over their sum; softmax 1: chosen by z + correction, weights the softmax over the chosen's (one group).
 EMBER_API int ember_moe_pick(const float* logits, int ld, const float* correction, int T, int experts, int top, int groups,
-                             int keep, float scale, int* chosen, float* weights, cudaStream_t stream) {
+                             int keep, float scale, int softmax, int* chosen, float* weights, cudaStream_t stream) {
+  EMBER_CHECK(!softmax || groups == 1, "moe_pick: a softmax over the chosen with %d groups", groups);
   EMBER_CHECK(T > 0 && experts > 0 && experts <= 1024 && top >= 1 && top <= experts && ld >= experts,
               "moe_pick: %d tokens, top %d of %d experts (at most 1024)", T, top, experts);
   EMBER_CHECK(groups >= 1 && experts % groups == 0 && keep >= 1 && keep <= groups && (long long)keep * (experts / groups) >= top,
               "moe_pick: %d groups of which %d are kept do not hold %d choices", groups, keep, top);
   const size_t smem = (size_t)kPickWarps * (2 * experts + groups) * sizeof(float);
   const cudaError_t e = launch_plain(moe_pick_kernel, dim3((T + kPickWarps - 1) / kPickWarps), dim3(32 * kPickWarps), smem, stream,
-                                     logits, ld, correction, T, experts, top, groups, keep, scale, chosen, weights);
+                                     logits, ld, correction, T, experts, top, groups, keep, scale, softmax, chosen, weights);
   if (e != cudaSuccess) return ember_fail("moe_pick: %s", cudaGetErrorString(e));
   return 0;
 }

@@ -34,7 +34,18 @@ _SIGNATURES = {
     "ember_generalized_delta_rule": [_c_void, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_float,
                                      _c_float, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void,
                                      _c_int, _c_void],
-    "ember_moe_pick": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void, _c_void, _c_void],
+    "ember_moe_pick": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void, _c_void, _c_void],
+    "ember_post_norm": [_c_void, _c_float, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_float, _c_float,
+                        _c_float, _c_void, _c_void, _c_void, _c_int, _c_void, _c_void, _c_int, _c_int, _c_void],
+    "ember_depth_average": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_size, _c_void],
+    "ember_qkv_prepare": [_c_void, ctypes.c_longlong, _c_void, ctypes.c_longlong, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
+                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_float, _c_int,
+                          _c_void, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void],
+    "ember_poly_norm": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void],
+    "ember_rglru": [_c_void, _c_void, _c_void, ctypes.c_longlong, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
+                    _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
+    "ember_rglru_step": [_c_void, _c_void, ctypes.c_longlong, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
+                         _c_int, _c_int, _c_int, _c_void],
     "ember_moe_combine": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_int, _c_int, _c_int, _c_void],
     "ember_moe_gate_up_act": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int,
                               _c_int, _c_int, _c_float, _c_float, _c_float, _c_void],
@@ -114,9 +125,9 @@ _SIGNATURES = {
     "ember_latent_rows": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int, _c_float, _c_void, _c_float, _c_int,
                           _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void],
     "ember_head_linear": [_c_void, ctypes.c_longlong, _c_int, _c_int, _c_void, _c_void, ctypes.c_longlong, _c_int, _c_int,
-                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
+                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ember_head_linear_bf16": [_c_void, ctypes.c_longlong, _c_int, _c_void, _c_void, ctypes.c_longlong, _c_int, _c_int, _c_int,
-                               _c_int, _c_int, _c_void, _c_size, _c_void],
+                               _c_int, _c_int, _c_int, _c_void, _c_size, _c_void],
     "ember_latent_attention_plain": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int,
                                      _c_int, _c_int, _c_int, _c_float, _c_int, _c_void],
     "ember_latent_attention_mma": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int,
@@ -211,8 +222,9 @@ def load_library() -> ctypes.CDLL:
     lib.ember_attention_decode_kept_scratch.restype = _c_size
     lib.ember_mlstm_scan_scratch.argtypes = [_c_int] * 5
     lib.ember_mlstm_scan_scratch.restype = _c_size
-    lib.ember_mingru_scratch.argtypes = [_c_int] * 3
-    lib.ember_mingru_scratch.restype = _c_size
+    for name in ("ember_mingru_scratch", "ember_rglru_scratch"):
+        getattr(lib, name).argtypes = [_c_int] * 3
+        getattr(lib, name).restype = _c_size
     for name in ("ember_tc_status", "ember_linear_decode_status", "ember_attention_decode_status",
                  "ember_attention_decode_mma_status"):
         getattr(lib, name).argtypes = []
@@ -1117,23 +1129,23 @@ class CudaOps:
 
     def head_linear(self, a, a_col, a_head, w, out, out_col, out_head):
         """out[t, out_col + h * out_head + (0..N)] = a[t, a_col + h * a_head + (0..K)] w[h]^T for every head h of
-        w [heads, N, K]; float32 sums."""
+        w [heads, N, K]; float32 sums, the output in the rows' element type or float32."""
         heads, N, K = w.shape
         T = a.shape[0]
-        if a.dtype != w.dtype or out.dtype != w.dtype or out.shape[0] != T or a.stride(1) != 1 or out.stride(1) != 1:
-            raise KernelError("head_linear: rows, matrices and output of one element type")
+        if a.dtype != w.dtype or out.dtype not in (w.dtype, torch.float32) or out.shape[0] != T or a.stride(1) != 1 or out.stride(1) != 1:
+            raise KernelError("head_linear: rows and matrices of one element type, the output of that type or float32")
         if a_col + (heads - 1) * a_head + K > a.shape[1] or out_col + (heads - 1) * out_head + N > out.shape[1]:
             raise KernelError("head_linear: the heads do not fit the rows")
         if w.dtype == torch.bfloat16 and T > SMALL_M and self.gemm == "lt":
             # the library's strided batch (a head's offset as the batch stride), where everything lies on 16 bytes
             ws = self._lt_workspace()
             rc = self._call("ember_head_linear_bf16", a.data_ptr() + 2 * int(a_col), a.stride(0), int(a_head),
-                            self._dense(w, "matrices").data_ptr(), out.data_ptr() + 2 * int(out_col), out.stride(0), int(out_head),
-                            T, heads, N, K, ws.data_ptr(), ws.numel(), allow=(2,))
+                            self._dense(w, "matrices").data_ptr(), out.data_ptr() + out.element_size() * int(out_col),
+                            out.stride(0), int(out_head), T, heads, N, K, _code(out.dtype), ws.data_ptr(), ws.numel(), allow=(2,))
             if rc == 0:
                 return out
         self._call("ember_head_linear", a.data_ptr(), a.stride(0), int(a_col), int(a_head), self._dense(w, "matrices").data_ptr(),
-                   out.data_ptr(), out.stride(0), int(out_col), int(out_head), T, heads, N, K, _code(w.dtype))
+                   out.data_ptr(), out.stride(0), int(out_col), int(out_head), T, heads, N, K, _code(w.dtype), _code(out.dtype))
         return out
 
     def latent_attention(self, rows, cache, plan, heads, kv_rank, rot_dim, scale, out_dtype):
@@ -1312,18 +1324,19 @@ class CudaOps:
             tiled = dtype == torch.bfloat16 and pairs >= MOE_TILE_PAIRS
         return 1 if tiled and k % 8 == 0 and n_out % 2 == 0 else 0
 
-    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale):
+    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale, softmax=False):
         """The router's choice for every row of float32 logits [T, >= experts]: scores sigmoid(z); chosen on score +
         correction among the experts of the `keep_groups` groups (of `groups` equal groups of neighbours) whose two
         largest choice scores add up to the most; weights = the chosen's scores over their sum (+ 1e-20) times
-        `route_scale`.  Returns (chosen int32 [T, top], weights float32 [T, top])."""
+        `route_scale`.  `softmax`: chosen on z + correction, weights = the softmax over the chosen's z + correction, times
+        `route_scale` (one group).  Returns (chosen int32 [T, top], weights float32 [T, top])."""
         T = logits.shape[0]
         if logits.dtype != torch.float32 or logits.shape[1] < experts or correction.dtype != torch.float32 or correction.numel() != experts:
             raise KernelError("moe_pick: float32 logits of at least `experts` columns and a float32 correction an expert")
         chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
         weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
         self._call("ember_moe_pick", self._dense(logits, "logits").data_ptr(), logits.shape[1], correction.data_ptr(), T, int(experts),
-                   int(top), int(groups), int(keep_groups), float(route_scale), chosen.data_ptr(), weights.data_ptr())
+                   int(top), int(groups), int(keep_groups), float(route_scale), 1 if softmax else 0, chosen.data_ptr(), weights.data_ptr())
         return chosen, weights
 
     def moe_combine(self, x, y, weights, shared, logits, gate_col):
@@ -1360,6 +1373,161 @@ class CudaOps:
         self._call("ember_moe_down", self._dense(inner_rows, "rows").data_ptr(), self._dense(w_down, "experts").data_ptr(),
                    pair_expert.data_ptr(), offsets.data_ptr(), order.data_ptr(), out.data_ptr(), T, top, experts, width,
                    inner, self._moe_tiled(T * top, inner_rows.dtype, tiled, inner, width), _code(inner_rows.dtype))
+        return out
+
+    # ------------------------------------------------------------------ norms after the sum, sums over depth
+    def _history(self, history, rows, d):
+        for t in history:
+            if t.dtype != torch.float32 or tuple(t.shape) != (rows, d) or not t.is_contiguous() or not t.is_cuda:
+                raise KernelError("depth average: every layer's result is a contiguous float32 tensor of the stream's shape")
+        return (_c_void * max(len(history), 1))(*[t.data_ptr() for t in history])
+
+    def post_norm(self, x, alpha, branches, w, eps, offset, dtype, branch_eps=0.0, history=None, coef=None):
+        """y = rmsnorm(alpha * x + sum of factor * b over `branches`) * (offset + w) in one launch.  A branch is (float32 rows,
+        factor) or (rows, factor, gain): with a gain the rows are divided by their root mean square (`branch_eps`) and
+        multiplied by it first; a factor may be float32 [rows], one a row.  With `history` (the results of the layers in
+        front, X_0 first) and `coef` (float32 [len(history) + 1]) the stream goes on as their weighted sum with y as the last.
+        Returns (y, stream, the stream's rows in `dtype`); without a history the stream is y, in float32 the rows are it."""
+        rows, d = x.shape
+        if x.dtype != torch.float32 or not x.is_contiguous() or w.dtype != torch.float32 or w.shape[0] != d:
+            raise KernelError("post_norm: a contiguous float32 stream and a float32 gain of its width")
+        n = len(branches)
+        if not 1 <= n <= 32:
+            raise KernelError(f"post_norm: {n} branches (1 to 32)")
+        factors, weights, gains = [], [], []
+        for b in branches:
+            t, f, g = b[0], b[1], (b[2] if len(b) > 2 else None)
+            if t.dtype != torch.float32 or tuple(t.shape) != (rows, d) or t.stride(1) != 1 or not t.is_cuda:
+                raise KernelError("post_norm: every branch is float32 [rows, width] with contiguous rows")
+            if g is not None and (g.dtype != torch.float32 or tuple(g.shape) != (d,)):
+                raise KernelError("post_norm: a branch's gain is float32 of the row's width")
+            if torch.is_tensor(f):
+                if f.dtype != torch.float32 or tuple(f.shape) != (rows,) or not f.is_cuda:
+                    raise KernelError("post_norm: factors a row are float32, one a row")
+                factors.append(1.0)
+                weights.append(f)
+            else:
+                factors.append(float(f))
+                weights.append(None)
+            gains.append(g)
+        if (history is None) != (coef is None) or (coef is not None and (coef.dtype != torch.float32 or coef.numel() != len(history) + 1)):
+            raise KernelError("post_norm: one float32 coefficient for every layer in front and one for this one")
+        y = torch.empty_like(x)
+        stream = y if history is None else torch.empty_like(x)
+        copy = None if dtype == torch.float32 else torch.empty((rows, d), dtype=dtype, device=x.device)
+        hist = None if history is None else self._history(history, rows, d)
+        self._call("ember_post_norm", x.data_ptr(), float(alpha), (_c_void * n)(*[b[0].data_ptr() for b in branches]),
+                   (ctypes.c_longlong * n)(*[b[0].stride(0) for b in branches]), (_c_float * n)(*factors),
+                   (_c_void * n)(*[self._ptr(t) for t in weights]), (_c_int * n)(*[0 if t is None else t.stride(0) for t in weights]),
+                   (_c_void * n)(*[self._ptr(g) for g in gains]), n, w.data_ptr(), float(offset), float(eps), float(branch_eps),
+                   y.data_ptr(), self._ptr(copy), hist, 0 if history is None else len(history), self._ptr(coef),
+                   None if history is None else stream.data_ptr(), rows, d)
+        return y, stream, stream if copy is None else copy
+
+    def depth_average(self, history, coef, dtype):
+        """(sum over j of coef[j] * history[j], the same in `dtype`): float32 tensors of one shape, float32 coefficients."""
+        rows, d = history[0].shape
+        if coef.dtype != torch.float32 or coef.numel() != len(history):
+            raise KernelError("depth_average: one float32 coefficient for every tensor")
+        stream = torch.empty_like(history[0])
+        copy = None if dtype == torch.float32 else torch.empty((rows, d), dtype=dtype, device=stream.device)
+        self._call("ember_depth_average", self._history(history, rows, d), len(history), coef.data_ptr(), stream.data_ptr(),
+                   self._ptr(copy), rows * d)
+        return stream, stream if copy is None else copy
+
+    def cast_rows(self, x, dtype):
+        """Float32 rows in the compute type (the same tensor in float32)."""
+        if dtype == torch.float32:
+            return x
+        out = torch.empty(x.shape, dtype=dtype, device=x.device)
+        self._call("ember_cast_rows", self._dense(x, "rows").data_ptr(), out.data_ptr(), x.numel(), _code(dtype))
+        return out
+
+    # ------------------------------------------------------------------ q, k and v between projection and attention
+    _QK_NORMS = {None: 0, "row": 1, "head": 2}
+
+    def qkv_prepare(self, proj, plan, cache, heads, kv_heads, head_dim, value_dim, out_dtype, store, v_col=None, norm=None,
+                    q_gain=None, k_gain=None, eps=0.0, rotary=None, unit_after=False):
+        """Norms, rotation and the cache's new rows in one launch, float32 in between: from rows q | k | v of `proj` (q alone
+        where `store` is False: the keys and values are another layer's), the query heads into rows of q | k | v (the
+        layout that `attention` reads; the rest of a row is not written) and the keys and values into the cache's
+        pages.  norm "row": q and k divided by their root mean square over the whole row of heads and multiplied by gains of its
+        width; "head": a head at a time, gains of the head's size (None: ones).  Then the rotation (a Rotary of
+        parts/position.py, or None), then with `unit_after` every q and k head divided by its own root mean square.  v_col: the
+        column the values start at (default: behind the keys; the keys' own column makes them the keys as projected)."""
+        T = plan.T
+        q_w, k_w = heads * head_dim, kv_heads * head_dim
+        if norm not in self._QK_NORMS:
+            raise KernelError(f"qkv_prepare: norm {norm!r}")
+        if proj.shape[0] != T or proj.stride(1) != 1:
+            raise KernelError("qkv_prepare: one row of contiguous values a token")
+        for name, g, width in (("q", q_gain, q_w), ("k", k_gain, k_w)):
+            if g is not None and (g.dtype != torch.float32 or g.numel() != (width if norm == "row" else head_dim)):
+                raise KernelError(f"qkv_prepare: the gain of {name} is float32 of the norm's width")
+        if store and (cache.k.dtype != out_dtype or tuple(cache.k.shape[1:]) != (kv_heads, 64, head_dim)
+                      or tuple(cache.v.shape[1:]) != (kv_heads, 64, value_dim)):
+            raise KernelError("qkv_prepare: the cache's pages do not have the mixer's head sizes or element type")
+        out = torch.empty((T, q_w + k_w + kv_heads * value_dim), dtype=out_dtype, device=proj.device)
+        pages = plan.pages[cache.group_index]
+        self._call("ember_qkv_prepare", proj.data_ptr(), proj.stride(0), out.data_ptr(), out.stride(0),
+                   cache.k.data_ptr() if store else None, cache.v.data_ptr() if store else None, plan.positions.data_ptr(),
+                   plan.token_seq.data_ptr(), plan.seq_slot.data_ptr(), pages.data_ptr(), plan.max_blocks, T, heads,
+                   kv_heads if store else 0, head_dim, value_dim, q_w, q_w + k_w if v_col is None else int(v_col),
+                   self._QK_NORMS[norm], self._ptr(q_gain), self._ptr(k_gain), float(eps), 1 if unit_after else 0,
+                   None if rotary is None else rotary.freqs.data_ptr(), 1.0 if rotary is None else float(rotary.magnitude),
+                   0 if rotary is None else int(rotary.dims), 1 if rotary is not None and rotary.interleaved else 0,
+                   _code(proj.dtype), _code(out_dtype))
+        return out
+
+    # ------------------------------------------------------------------ PolyNorm
+    def poly_norm(self, z, four, eps, out_dtype):
+        """a N(z) + b N(z^2) + c N(z^3) + e over rows, N dividing a row by its root mean square; four = (a, b, c, e) float32."""
+        if four.dtype != torch.float32 or four.numel() != 4:
+            raise KernelError("poly_norm: four float32 numbers")
+        out = torch.empty(z.shape, dtype=out_dtype, device=z.device)
+        self._call("ember_poly_norm", self._dense(z, "rows").data_ptr(), out.data_ptr(), four.data_ptr(), z.shape[0], z.shape[1],
+                   float(eps), _code(z.dtype), _code(out_dtype))
+        return out
+
+    # ------------------------------------------------------------------ the real-gated linear recurrent unit
+    def rglru(self, u, proj, y_col, w_gates, bias_r, bias_i, rate, state, plan, pieces=None, one_launch=None):
+        """The recurrence of parts/rglru.py over the step's sequences: u [T, width], the output branch's columns from y_col
+        of `proj`, w_gates [parts, 2 * n, n] (a part's first gate, then its second), biases and rate float32 [width], state
+        float32 [slots, width] (advanced); S_t * gelu_tanh(y_t) in u's element type.  one_launch: the gates' products and the
+        recurrence as one launch (bfloat16 steps of one token a sequence; None lets the step decide)."""
+        T, width = u.shape
+        parts, n2, n = w_gates.shape
+        if u.dtype != w_gates.dtype or proj.dtype != u.dtype or parts * n != width or n2 != 2 * n or y_col + width > proj.shape[1]:
+            raise KernelError("rglru: u, the output branch and the gates' matrices of one element type and fitting sizes")
+        if state.dtype != torch.float32 or tuple(state.shape[1:]) != (width,) or any(
+                t.dtype != torch.float32 or t.numel() != width for t in (bias_r, bias_i, rate)):
+            raise KernelError("rglru: float32 state [slots, width], biases and rate [width]")
+        out = torch.empty((T, width), dtype=u.dtype, device=u.device)
+        y = proj[:, y_col:]
+        if one_launch is None:
+            one_launch = u.dtype == torch.bfloat16 and plan.all_single and T == plan.n
+        if one_launch:
+            rc = self._call("ember_rglru_step", self._dense(u, "u").data_ptr(), y.data_ptr(), proj.stride(0),
+                            self._dense(w_gates, "gates").data_ptr(), bias_r.data_ptr(), bias_i.data_ptr(), rate.data_ptr(),
+                            state.data_ptr(), out.data_ptr(), plan.seq_slot.data_ptr(), plan.seq_start.data_ptr(), T, width, parts,
+                            allow=(2,))
+            if rc == 0:
+                return out
+        gates = torch.empty((T, 2 * width), dtype=torch.float32, device=u.device)
+        self.head_linear(u, 0, n, w_gates, gates, 0, 2 * n)
+        longest = max(int(plan.max_new), 1)
+        if pieces is None:
+            pieces = self._pieces(longest, plan.n * -(-width // 128))
+        piece = -(-longest // pieces)
+        scratch = None
+        if pieces > 1:
+            scratch = torch.empty(self.lib.ember_rglru_scratch(plan.n, pieces, width), dtype=torch.float32, device=u.device)
+        self._call("ember_rglru", gates.data_ptr(), self._dense(u, "u").data_ptr(), y.data_ptr(), proj.stride(0), bias_r.data_ptr(),
+                   bias_i.data_ptr(), rate.data_ptr(), state.data_ptr(), out.data_ptr(), plan.seq_slot.data_ptr(),
+                   plan.seq_start.data_ptr(), plan.cu_new.data_ptr(), plan.n, width, parts, piece, pieces, self._ptr(scratch),
+                   _code(u.dtype))
+        if pieces > 1:
+            self.launches += 2
         return out
 
     # ------------------------------------------------------------------ sampling

@@ -81,6 +81,16 @@ class StepContext:
     position: object
     next_weights: tuple = ()   # set by the model: the first matrix that the block after the current one streams
     model_state: dict = dataclasses.field(default_factory=dict)   # per-sequence state of the parts in front of the layers
+    history: list = dataclasses.field(default_factory=list)       # results of the layers so far, where a layer sums over them
+    noted: tuple = (None, None)                                   # a float32 stream and its rows in the compute type
+
+    def note_rows(self, stream, rows) -> None:
+        """Keeps the rows in the compute type that a launch wrote beside the float32 stream."""
+        self.noted = (stream, rows)
+
+    def rows_of(self, stream):
+        """The stream's rows in the compute type: noted ones, or a conversion."""
+        return self.noted[1] if self.noted[0] is stream else self.ops.cast_rows(stream, self.dtype)
 
 
 class Engine:

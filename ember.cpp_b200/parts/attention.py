@@ -35,6 +35,14 @@ mixer rotates the first `dims` dimensions of every q and k head itself, neighbou
 `interleaved`; `head_scale`: the name of one learned factor a query head on its scores; `chunk` = size: query i
 sees key j <= i only if floor(i / size) = floor(j / size), counted from the sequence's position 0 (the cache
 then keeps the pages of the query's own run alone); `fixed_sink` = s: a sink whose score is the constant s.
+
+And: `qk_norm_scope` = "head": the norms of `qk_norm` are a head at a time, with one gain of the head's size for all
+heads; `unit_qk`: after the rotation every q and k head is divided by its own root mean square (no gain); `rotary` may
+carry a fourth entry, the frequencies' scaling (parts/position.py); `values_are_keys`: the values are the keys as
+projected (biases included), before norm and rotation, and there is no value matrix; `shares_cache`: the layer has no
+tensors of keys and values and reads the keys and values that another entry of the schedule cached.  With any of these,
+or with both norms and a rotation, the projection stays in float32 and one launch makes norms and rotation of q and
+k, rounds once, and puts keys and values straight into the cache's pages (`ops.qkv_prepare`).
 """
 from __future__ import annotations
 
@@ -53,7 +61,8 @@ class CausalAttention(Mixer):
                  keep_first: int = 0, value_dim: int | None = None, suffix: str = ".weight", qk_norm=None,
                  value_norm: bool = False, norm_eps: float = 0.0, q_temp=None, distance_slope_base: float | None = None,
                  sink: str | None = None, gate: str | None = None, qkv_bias: str | None = None, conv=None, rotary=None,
-                 head_scale: str | None = None, chunk: int = 0, fixed_sink: float | None = None):
+                 head_scale: str | None = None, chunk: int = 0, fixed_sink: float | None = None, qk_norm_scope: str = "row",
+                 unit_qk: bool = False, values_are_keys: bool = False, shares_cache: bool = False):
         super().__init__(prefix)
         if n_heads % kv_heads:
             raise ValueError(f"attention {prefix!r}: {n_heads} heads are not a multiple of {kv_heads} key/value heads")
@@ -82,7 +91,8 @@ class CausalAttention(Mixer):
         self.rotary = None
         if rotary is not None:
             from .position import Rotary
-            self.rotary = Rotary(prefix, dims=int(rotary[0]), base=float(rotary[1]), interleaved=bool(rotary[2]))
+            self.rotary = Rotary(prefix, dims=int(rotary[0]), base=float(rotary[1]), interleaved=bool(rotary[2]),
+                                 scaling=rotary[3] if len(rotary) > 3 else None)
             if self.rotary.dims > head_dim:
                 raise ValueError(f"attention {prefix!r}: {self.rotary.dims} rotated dimensions of a head of {head_dim}")
         if self.chunk < 0 or (self.chunk and window):
@@ -94,11 +104,24 @@ class CausalAttention(Mixer):
         if (qkv_bias is not None or self.conv is not None) and (isinstance(qkv, str) or bias):
             raise ValueError(f"attention {prefix!r}: biases on q, k and v alone and convolutions come with q, k and v "
                              "stored as three matrices, without the fused projection's biases")
+        if qk_norm_scope not in ("row", "head"):
+            raise ValueError(f"attention {prefix!r}: qk_norm_scope = {qk_norm_scope!r}")
+        self.qk_norm_scope, self.unit_qk = qk_norm_scope, bool(unit_qk)
+        self.values_are_keys, self.shares_cache = bool(values_are_keys), bool(shares_cache)
+        # norms and a rotation together, or what only the one launch of both knows
+        self.one_prepare = (self.unit_qk or self.values_are_keys or self.shares_cache or
+                            (self.qk_norm_names is not None and (qk_norm_scope == "head" or self.rotary is not None)))
+        if self.one_prepare and (isinstance(qkv, str) or bias or self.value_norm or self.q_temp is not None or self.gate_name is not None
+                                 or self.conv is not None):
+            raise ValueError(f"attention {prefix!r}: norms a head, norms with a rotation, values that are keys and another entry's "
+                             "cache come with q, k and v stored apart, without value norms, temperatures, gates or convolutions")
+        if self.values_are_keys and value_dim is not None and int(value_dim) != int(head_dim):
+            raise ValueError(f"attention {prefix!r}: values that are the keys have the keys' size, not {value_dim}")
         self.biased = (self.slope_base is not None or self.sink_name is not None or self.fixed_sink is not None
                        or self.chunk > 0 or self.head_scale_name is not None)
-        if (self.prepared or slope_base_or_sink(distance_slope_base, sink)) and bias:
+        if (self.prepared or self.one_prepare or slope_base_or_sink(distance_slope_base, sink)) and bias:
             raise ValueError(f"attention {prefix!r}: norms, gates, slopes and sinks come without biases")
-        self.extended = int(keep_first) > 0 or value_dim is not None or self.prepared or self.biased
+        self.extended = int(keep_first) > 0 or value_dim is not None or self.prepared or self.biased or self.one_prepare
         self.value_dim = self.head_dim if value_dim is None else int(value_dim)
         if not 1 <= self.value_dim <= 256:
             raise ValueError(f"attention {prefix!r}: value size {self.value_dim} is not in [1, 256]")
@@ -120,10 +143,14 @@ class CausalAttention(Mixer):
     def _shape(self, n_in, n_out):
         return (n_in, n_out) if self.stored == "in_out" else (n_out, n_in)
 
+    def _projections(self):
+        """(name, output width) of the matrices that the layer has of q, k and v stored apart."""
+        return list(zip(self.qkv_name, self.widths))[:1 if self.shares_cache else (2 if self.values_are_keys else 3)]
+
     def weight_specs(self):
         if self.split:
             specs = [WeightSpec(n + self.suffix, self._shape(self.width, w), std=self.init_std)
-                     for n, w in zip(self.qkv_name, self.widths)]
+                     for n, w in self._projections()]
         else:
             specs = [WeightSpec(self.qkv_name + self.suffix, self._shape(self.width, self.qkv_width), std=self.init_std)]
         specs.append(WeightSpec(self.out_name + self.suffix, self._shape(self.o_width, self.width), std=self.out_init_std))
@@ -131,14 +158,15 @@ class CausalAttention(Mixer):
             specs += [WeightSpec(self.qkv_name + ".bias", (self.qkv_width,), std=self.bias_init_std),
                       WeightSpec(self.out_name + ".bias", (self.width,), std=self.bias_init_std)]
         if self.qk_norm_names is not None:
-            specs += [WeightSpec(self.qk_norm_names[0], (self.q_width,), mean=1.0, std=0.1),
-                      WeightSpec(self.qk_norm_names[1], (self.widths[1],), mean=1.0, std=0.1)]
+            per_head = self.qk_norm_scope == "head"
+            specs += [WeightSpec(n, (self.head_dim if per_head else w,), mean=1.0, std=0.1)
+                      for n, w in list(zip(self.qk_norm_names, self.widths))[:1 if self.shares_cache else 2]]
         if self.sink_name is not None:
             specs.append(WeightSpec(self.sink_name, (self.n_heads,), std=1.0))
         if self.gate_name is not None:
             specs.append(WeightSpec(self.gate_name + self.suffix, self._shape(self.width, self.o_width), std=self.init_std))
         if self.qkv_bias_suffix is not None:
-            specs += [WeightSpec(n + self.qkv_bias_suffix, (w,), std=self.bias_init_std * 10) for n, w in zip(self.qkv_name, self.widths)]
+            specs += [WeightSpec(n + self.qkv_bias_suffix, (w,), std=self.bias_init_std * 10) for n, w in self._projections()]
         if self.conv is not None:
             specs += [WeightSpec(n + self.conv[1], (w, self.conv[0]), std=0.5) for n, w in zip(self.qkv_name, self.widths)]
         if self.head_scale_name is not None:
@@ -154,7 +182,7 @@ class CausalAttention(Mixer):
                              "the float32 path takes this model")
         t = self.stored == "in_out"
         if self.split:
-            self.w_qkv = torch.cat([runtime.matrix(get(n + self.suffix), transpose=t) for n in self.qkv_name]).contiguous()
+            self.w_qkv = torch.cat([runtime.matrix(get(n + self.suffix), transpose=t) for n, _ in self._projections()]).contiguous()
         else:
             self.w_qkv = runtime.matrix(get(self.qkv_name + self.suffix), transpose=t)
         self.w_out = runtime.matrix(get(self.out_name + self.suffix), transpose=t)
@@ -163,7 +191,8 @@ class CausalAttention(Mixer):
             pad = torch.zeros((self.gate_col - self.qkv_width, self.width), dtype=self.w_qkv.dtype, device=self.w_qkv.device)
             self.w_qkv = torch.cat([self.w_qkv, pad, runtime.matrix(get(self.gate_name + self.suffix), transpose=t)]).contiguous()
         if self.qk_norm_names is not None:
-            self.q_gain, self.k_gain = (runtime.vector(get(n)) for n in self.qk_norm_names)
+            self.q_gain = runtime.vector(get(self.qk_norm_names[0]))
+            self.k_gain = None if self.shares_cache else runtime.vector(get(self.qk_norm_names[1]))
         if self.sink_name is not None:
             self.sinks = runtime.vector(get(self.sink_name))
         if self.slope_base is not None:
@@ -173,7 +202,7 @@ class CausalAttention(Mixer):
             self.b_qkv = runtime.vector(get(self.qkv_name + ".bias"))
             self.b_out = runtime.vector(get(self.out_name + ".bias"))
         if self.qkv_bias_suffix is not None:
-            self.b_qkv = torch.cat([runtime.vector(get(n + self.qkv_bias_suffix)) for n in self.qkv_name]).contiguous()
+            self.b_qkv = torch.cat([runtime.vector(get(n + self.qkv_bias_suffix)) for n, _ in self._projections()]).contiguous()
         if self.conv is not None:
             self.conv_w = torch.cat([runtime.vector(get(n + self.conv[1])) for n in self.qkv_name]).contiguous()
             self.conv_b = torch.zeros(self.qkv_width, dtype=torch.float32, device=self.conv_w.device)
@@ -204,8 +233,35 @@ class CausalAttention(Mixer):
         return CacheNeed("window" if windowed else "full", self.kv_heads, self.head_dim, self.window,
                          self.keep_first if windowed else 0, 0 if self.value_dim == self.head_dim else self.value_dim)
 
+    def _attend_prepared(self, ctx, h, app):
+        import torch
+        ops = ctx.ops
+        if app.writes_cache == self.shares_cache:
+            raise ValueError(f"attention {self.prefix!r}: a layer with keys and values of its own writes the cache, a layer "
+                             "without them reads another entry's")
+        proj = ops.linear(h, self.w_qkv, self.b_qkv, out_dtype=torch.float32)            # float32 [T, q (| k (| v))]
+        norm = None if self.qk_norm_names is None else self.qk_norm_scope
+        qkv = ops.qkv_prepare(proj, ctx.plan, app.cache, self.n_heads, self.kv_heads, self.head_dim, self.value_dim, ctx.dtype,
+                              store=not self.shares_cache, v_col=self.q_width if self.values_are_keys else None, norm=norm,
+                              q_gain=self.q_gain, k_gain=self.k_gain, eps=self.norm_eps, rotary=self.rotary, unit_after=self.unit_qk)
+        more = dict(slopes=self.slopes, sinks=self.sinks, chunk=self.chunk, head_scales=self.head_scales,
+                    head_scales_positive=self.head_scales is None or self.head_scales_positive)
+        if self._plain_sight(ctx.dtype):
+            return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
+                                 out_dtype=ctx.dtype, store=False)
+        return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
+                             out_dtype=ctx.dtype, store=False, keep_first=self.keep_first if self.window > 0 else 0,
+                             value_dim=self.value_dim, **more)
+
+    def _plain_sight(self, dtype) -> bool:
+        """Nothing but a window on the scores, and sizes that the kernels for such heads have."""
+        return (not self.biased and self.keep_first == 0 and self.value_dim == self.head_dim and self.head_dim in (64, 128)
+                and self.n_heads // self.kv_heads <= 8 and self.scale > 0)
+
     def _attend(self, ctx, h, app):
         ops = ctx.ops
+        if self.one_prepare:
+            return self._attend_prepared(ctx, h, app)
         if self.prepared:
             import torch
             proj = ops.linear(h, self.w_qkv, None, out_dtype=torch.float32)          # float32 [T, q | k | v (| 0 | g)]

@@ -6,6 +6,7 @@ tensors are named by a prefix that the architecture gives it.  No part knows whi
 Roles and what each must provide:
 
   norm      forward(ctx, x, out_dtype) -> tensor                     (x: fp32 residual stream)
+            sum_normed(ctx, x, alpha, branches) -> new stream        (for arrangements that norm after the sum)
   mixer     forward(ctx, h, residual, app) -> new residual stream    (h: normed input)
             cache_need() -> CacheNeed | None, state_need() -> StateNeed | {name: StateNeed} | None
   ffn       forward(ctx, h, residual) -> new residual stream
@@ -14,13 +15,14 @@ Roles and what each must provide:
             a norm's add_normed(ctx, x, branches) makes that sum, norms it and adds it to the stream.  A branch
             may carry a third entry (gain, eps): its rows are then divided by their root mean square and
             multiplied by that gain before they are weighted; `plain_branches` does that for a consumer that has
-            no kernel for it)
+            no kernel for it; `row_branches(ctx, h)` of a feed-forward may give factors that are tensors, one a row)
   embed     forward(ctx, x, state) -> x     (adds to the embedded rows; state_need() as a mixer's: what it
             carries per sequence, kept by the cache beside the layers' states)
   position  embedding_table() -> tensor | None, max_positions() -> int | None,
             apply_qk(ctx, qkv, n_heads, kv_heads, head_dim) (in place; default: nothing)
   addon     forward(ctx, x) -> x            (something added to the stream after a layer's sublayers, reading the
-            stream itself and, where it sets `needs_tokens`, the step's token ids)
+            stream itself and, where it sets `needs_tokens`, the step's token ids; with `reads_history` it finds the
+            results of the layers in front in `ctx.history`)
   block     forward(ctx, x, app) -> x       (the arrangement of the parts above)
 
 Every part lists its tensors with `weight_specs()` (name, stored shape, how random-weights mode
@@ -64,6 +66,18 @@ class CacheNeed:
     @property
     def v_dim(self) -> int:
         return self.value_dim or self.head_dim
+
+    def joined(self, other: "CacheNeed") -> "CacheNeed":
+        """The least need that serves both (a layer's own mixer and one that reads its cache): the wider window, or all
+        keys where the two limit sight in different ways."""
+        if (self.kv_heads, self.head_dim, self.v_dim) != (other.kv_heads, other.head_dim, other.v_dim):
+            raise ValueError(f"a cache of {self.kv_heads} heads of {self.head_dim} and {self.v_dim} values is read as "
+                             f"{other.kv_heads} of {other.head_dim} and {other.v_dim}")
+        if self == other:
+            return self
+        if self.kind == other.kind == "window":
+            return dataclasses.replace(self, window=max(self.window, other.window), keep_first=max(self.keep_first, other.keep_first))
+        return dataclasses.replace(self, kind="full", window=0, keep_first=0)
 
 
 @dataclasses.dataclass(frozen=True)
@@ -127,6 +141,15 @@ class Norm(Part):
             total = term if total is None else total + term
         return x + self.forward(ctx, total.contiguous(), x.dtype)
 
+    def sum_normed(self, ctx, x, alpha, branches, average=None):
+        """norm(alpha * x + sum of factor * rows over `branches`) as a new float32 stream; `average`: a DepthAverage that
+        follows at once, whose sum is then the stream.  A norm whose kernel does all of it in one launch overrides this."""
+        total = x * alpha
+        for rows, factor in plain_branches(ctx, branches):
+            total = total + rows.float() * (factor[:, None] if hasattr(factor, "dim") else factor)
+        y = self.forward(ctx, total.contiguous(), x.dtype)
+        return y if average is None else average.forward(ctx, y)
+
 
 class Mixer(Part):
     role = "mixer"
@@ -163,6 +186,10 @@ class FeedForward(Part):
         zero = torch.zeros((h.shape[0], self.width), dtype=torch.float32, device=h.device)
         return [(self.forward(ctx, h, zero), 1.0)]
 
+    def row_branches(self, ctx, h):
+        """`branches` for a caller that takes factors of their own for every row (float32 [T] tensors) as well."""
+        return self.branches(ctx, h)
+
 
 class EmbedPart(Part):
     """Something added to the embedded rows before the first layer (rows of a second table chosen by more
@@ -182,6 +209,7 @@ class StreamAddon(Part):
     token ids, for instance).  It reads the float32 stream and returns the new one."""
     role = "addon"
     needs_tokens = False
+    reads_history = False
 
     def forward(self, ctx, x):
         raise NotImplementedError
@@ -202,6 +230,7 @@ class Position(Part):
 
 class Block(Part):
     role = "block"
+    in_place = True      # False: the arrangement never adds into the stream that it is given
 
     def __init__(self, norm1: "Norm | None", mixer: Mixer, norm2: "Norm | None", ffn: "FeedForward | None", **more_norms: Norm):
         super().__init__("")
@@ -244,8 +273,8 @@ def build_part(role: str, spec: PartSpec) -> Part:
     return kinds[spec.kind](prefix=spec.prefix, **spec.params)
 
 
-def build_block(kind: str, norm1, mixer, norm2, ffn, more_norms=None) -> Block:
+def build_block(kind: str, norm1, mixer, norm2, ffn, more_norms=None, params=None) -> Block:
     kinds = _REGISTRY["block"]
     if kind not in kinds:
         raise ValueError(f"no block arrangement {kind!r} is registered; registered: {registered('block')}")
-    return kinds[kind](norm1, mixer, norm2, ffn, **(more_norms or {}))
+    return kinds[kind](norm1, mixer, norm2, ffn, **(more_norms or {}), **(params or {}))

@@ -16,6 +16,12 @@ arrangement may have no feed-forward; it then has no norms around one either.
 `shared_norm` has one norm that both sublayers read: `h = norm1(x)`, `x -> x + mixer(h) + ffn(h)`.
 The mixer's last projection adds into the stream and the feed-forward's adds into that, both in
 float32; a layer of this arrangement may have no feed-forward.
+
+`post_norm` norms after the sum: `x -> norm1(alpha * x + mixer(x))`, then `x -> norm2(alpha * x + ffn(x))`, alpha a
+constant (DeepNorm: Wang et al., "DeepNet: Scaling Transformers to 1,000 Layers").  The sublayers read the stream
+itself, in the compute type; they hand over their outputs as branches and the norm's launch makes the sum, the norm, the
+rows in the compute type and, where the layer's first addon is a sum over depth, that sum too.  A layer of this
+arrangement may have no feed-forward and then has no second norm.
 """
 from __future__ import annotations
 
@@ -81,6 +87,32 @@ class SharedNormBlock(Block):
         return x if self.ffn is None else self.ffn.forward(ctx, h, x)
 
 
+class PostNormBlock(Block):
+    in_place = False
+
+    def __init__(self, norm1, mixer, norm2, ffn, alpha: float = 1.0, **more_norms):
+        if norm1 is None or more_norms or (ffn is None) != (norm2 is None):
+            raise ValueError("block 'post_norm' has a norm after the mixer's sum and, with a feed-forward, one after that's")
+        super().__init__(norm1, mixer, norm2, ffn)
+        self.alpha = float(alpha)
+
+    def forward(self, ctx, x, app):
+        announce = getattr(ctx.ops, "announce_weights", None)
+        if announce is not None:
+            announce(self.mixer.stream_weights() + (self.ffn.stream_weights() if self.ffn is not None else [])
+                     + list(getattr(ctx, "next_weights", ())))
+        addons = list(self.addons)
+        average = addons.pop(0) if addons and addons[0].reads_history else None
+        branches = self.mixer.branches(ctx, ctx.rows_of(x), app)
+        x = self.norm1.sum_normed(ctx, x, self.alpha, branches, average if self.ffn is None else None)
+        if self.ffn is not None:
+            x = self.norm2.sum_normed(ctx, x, self.alpha, self.ffn.row_branches(ctx, ctx.rows_of(x)), average)
+        for part in addons:
+            x = part.forward(ctx, x)
+        return x
+
+
+register_part("block", "post_norm", PostNormBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "shared_norm", SharedNormBlock)
 register_part("block", "sandwich", SandwichBlock)

@@ -5,6 +5,9 @@ ember.cpp's GPT-2 block: `u = h Wup^T + b; u = gelu(u); f = u Wdown^T + b; x = x
 `0.5 v (1 + tanh(sqrt(2/pi) (v + 0.044715 v^3)))` or its erf form `0.5 v (1 + erf(v / sqrt 2))`
 (graph_ir.cpp:2471-2481; graph_ir_cuda.cu:230-242).
 
+`poly_norm`: an activation of whole rows, a N(u) + b N(u^2) + c N(u^3) + e with four learned numbers and N the division of
+a row by its root mean square (float32 arithmetic, csrc/poly_norm.cu).
+
 Gated feed-forward: two projections of the input side by side, `y = act(g) * u`, then the down
 projection.  `silu`: act(g) = g * sigmoid(g), the usual gated layer.  `clamped_sigmoid`: g is first
 capped from above at `limit` and u held within +-`limit`, then y = g * sigmoid(alpha * g) * (u + shift).
@@ -15,18 +18,23 @@ from __future__ import annotations
 from .base import FeedForward, WeightSpec, register_part
 
 ACTIVATIONS = ("gelu_tanh", "gelu_erf", "relu2")     # relu2: the square of relu
+ROW_ACTIVATIONS = ("poly_norm",)                      # activations with weights of their own that see a whole row
 
 
 class DenseFeedForward(FeedForward):
 
     def __init__(self, prefix: str, width: int, inner: int, activation: str, up: str = "c_fc", down: str = "c_proj",
                  stored: str = "in_out", bias: bool = True, init_std: float = 0.02, down_init_std: float = 0.02,
-                 bias_init_std: float = 0.01, suffix: str = ".weight", any_size: bool = False):
+                 bias_init_std: float = 0.01, suffix: str = ".weight", any_size: bool = False, act: str = "act",
+                 act_eps: float = 0.0):
+        """act, act_eps: the tensor of a row activation's own weights and the eps of its norms."""
         super().__init__(prefix)
         self.any_size = any_size  # True: widths that are no multiples of 8 are left to the slower products in bfloat16
         self.suffix = suffix      # what follows a matrix's name in the checkpoint ("" for names without one)
-        if activation not in ACTIVATIONS:
-            raise ValueError(f"feed-forward {prefix!r}: activation {activation!r} is not one of {ACTIVATIONS}")
+        if activation not in ACTIVATIONS + ROW_ACTIVATIONS:
+            raise ValueError(f"feed-forward {prefix!r}: activation {activation!r} is not one of {ACTIVATIONS + ROW_ACTIVATIONS}")
+        self.act_name, self.act_eps = (prefix + act, float(act_eps)) if activation in ROW_ACTIVATIONS else (None, 0.0)
+        self.act_w = None
         if stored not in ("in_out", "out_in"):
             raise ValueError(f"feed-forward {prefix!r}: stored = {stored!r}")
         self.width, self.inner, self.activation = int(width), int(inner), activation
@@ -43,6 +51,8 @@ class DenseFeedForward(FeedForward):
         if self.bias:
             specs += [WeightSpec(self.up_name + ".bias", (self.inner,), std=self.bias_init_std),
                       WeightSpec(self.down_name + ".bias", (self.width,), std=self.bias_init_std)]
+        if self.act_name is not None:
+            specs.append(WeightSpec(self.act_name, (4,), mean=0.3, std=0.2))
         return specs
 
     def load(self, get, runtime):
@@ -56,6 +66,8 @@ class DenseFeedForward(FeedForward):
         if self.bias:
             self.b_up = runtime.vector(get(self.up_name + ".bias"))
             self.b_down = runtime.vector(get(self.down_name + ".bias"))
+        if self.act_name is not None:
+            self.act_w = runtime.vector(get(self.act_name))
 
     def stream_weights(self):
         return [self.w_up, self.w_down]
@@ -64,12 +76,17 @@ class DenseFeedForward(FeedForward):
         warm = getattr(ctx.ops, "warm", None)
         if warm is not None:
             warm(self.w_down)  # a hint: the second product's weights can be on their way during the first
-        u = ctx.ops.linear(h, self.w_up, self.b_up, act=self.activation, out_dtype=ctx.dtype)
+        u = self._inner(ctx, h)
         return ctx.ops.linear(u, self.w_down, self.b_down, residual=residual)
+
+    def _inner(self, ctx, h):
+        if self.act_name is None:
+            return ctx.ops.linear(h, self.w_up, self.b_up, act=self.activation, out_dtype=ctx.dtype)
+        return ctx.ops.poly_norm(ctx.ops.linear(h, self.w_up, self.b_up, out_dtype=ctx.dtype), self.act_w, self.act_eps, ctx.dtype)
 
     def branches(self, ctx, h):
         import torch
-        u = ctx.ops.linear(h, self.w_up, self.b_up, act=self.activation, out_dtype=ctx.dtype)
+        u = self._inner(ctx, h)
         return [(ctx.ops.linear(u, self.w_down, self.b_down, out_dtype=torch.float32), 1.0)]
 
 

@@ -25,7 +25,8 @@ class DecoderModel:
         for layer in spec.layers:
             norm = lambda part: None if part is None else build_part("norm", part)  # noqa: E731
             self.blocks.append(build_block(layer.block, norm(layer.norm1), build_part("mixer", layer.mixer), norm(layer.norm2),
-                                           None if layer.ffn is None else build_part("ffn", layer.ffn), {name: norm(part) for name, part in layer.more_norms}))
+                                           None if layer.ffn is None else build_part("ffn", layer.ffn), {name: norm(part) for name, part in layer.more_norms},
+                                           layer.block_params))
             self.blocks[-1].addons = [build_part("addon", part) for part in layer.addons]
         self.final_norm = build_part("norm", spec.final_norm)
         self.embed_parts = [build_part("embed", part) for part in spec.embed_parts]
@@ -33,6 +34,7 @@ class DecoderModel:
         self.table = None
         self.head = None
         self.head_bias = None
+        self.keeps_history = any(getattr(p, "reads_history", False) for b in self.blocks for p in b.addons)
         self.reads_tokens = any(getattr(p, "needs_tokens", False) for p in self.all_parts())
 
     # ------------------------------------------------------------------ tensors
@@ -73,13 +75,14 @@ class DecoderModel:
 
     def application_needs(self):
         """(cache need, state need) of each entry of the schedule; an entry that reads another's
-        cache has no cache need of its own."""
-        out = []
-        for app in self.spec.schedule:
-            mixer = self.blocks[app.layer].mixer
-            need = None if app.cache_of is not None else mixer.cache_need()
-            out.append((need, mixer.state_need()))
-        return out
+        cache has no cache need of its own, but that cache must hold what it reads as well."""
+        mixers = [self.blocks[app.layer].mixer for app in self.spec.schedule]
+        needs = [None if app.cache_of is not None else m.cache_need() for app, m in zip(self.spec.schedule, mixers)]
+        for app, m in zip(self.spec.schedule, mixers):
+            read = None if app.cache_of is None else m.cache_need()
+            if read is not None and needs[app.cache_of] is not None:
+                needs[app.cache_of] = needs[app.cache_of].joined(read)
+        return [(need, m.state_need()) for need, m in zip(needs, mixers)]
 
     def model_state_needs(self) -> dict:
         """Per-sequence state that belongs to no layer: what the parts in front of the first layer carry,
@@ -124,6 +127,8 @@ class DecoderModel:
             x = part.forward(ctx, x, self._embed_state(ctx, i, part))
         if self.embed_norm is not None:
             x = self.embed_norm.forward(ctx, x, torch.float32)
+        if self.keeps_history:      # (a copy where the first layer would add into it)
+            ctx.history = [x.clone() if ctx.apps and self.blocks[ctx.apps[0].layer].in_place else x]
         for i, app in enumerate(ctx.apps):
             # (a hint for the kernels: the first matrix that the block after this one streams)
             following = ctx.apps[i + 1].layer if i + 1 < len(ctx.apps) else None

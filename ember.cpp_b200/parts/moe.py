@@ -93,6 +93,8 @@ class RoutedExperts(FeedForward):
     with `limit` > 0 the clamped form (g capped at limit, u within +-limit, g * sigmoid(alpha g) * (u + shift)).
     An optional shared expert of the same form (sizes and limit of its own) runs for every token and is added,
     multiplied by sigmoid(w_sg . h), one number a token, where `shared_gate` names w_sg.
+    With `scores` "softmax" the stored vector is a bias of the logits: the `top` largest of z + bias are chosen and weigh
+    the softmax over the chosen ones alone (times `route_scale`); experts are then in one group.
 
     The router's rows and the shared expert's gate row are one product with float32 sums; scores, choice,
     weights and the weighted sum are float32.  Nothing returns to the host."""
@@ -100,7 +102,7 @@ class RoutedExperts(FeedForward):
     def __init__(self, prefix: str, width: int, experts: int, top: int, inner: int, route_scale: float = 1.0,
                  groups: int = 1, keep_groups: int = 1, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
                  shared_inner: int = 0, shared_limit: float = 0.0, shared_gate: str | None = None,
-                 router: str = "router", correction: str | None = "correction", expert: str = "e{}.", shared: str = "shared.",
+                 scores: str = "sigmoid", router: str = "router", correction: str | None = "correction", expert: str = "e{}.", shared: str = "shared.",
                  gate: str = "gate", up: str = "up", down: str = "down", suffix: str = "", init_std: float = 0.02,
                  down_init_std: float = 0.02):
         super().__init__(prefix)
@@ -114,6 +116,9 @@ class RoutedExperts(FeedForward):
         if self.keep_groups * (self.experts // self.groups) < self.top:
             raise ValueError(f"experts {prefix!r}: {self.keep_groups} groups of {self.experts // self.groups} hold fewer "
                              f"than top = {self.top} experts")
+        if scores not in ("sigmoid", "softmax") or (scores == "softmax" and self.groups != 1):
+            raise ValueError(f"experts {prefix!r}: scores = {scores!r} with {self.groups} groups")
+        self.softmax = scores == "softmax"
         self.router_name = prefix + router
         self.correction_name = None if correction is None else prefix + correction
         self.expert_names = [tuple(prefix + expert.format(e) + n + suffix for n in (gate, up, down)) for e in range(self.experts)]
@@ -165,7 +170,7 @@ class RoutedExperts(FeedForward):
     def _chosen(self, ctx, h, logits):
         ops = ctx.ops
         chosen, weights = ops.moe_pick(logits, self.correction, self.experts, self.top, self.groups, self.keep_groups,
-                                       self.route_scale)
+                                       self.route_scale, **({"softmax": True} if self.softmax else {}))
         routing = ops.moe_route(None, ctx.plan.T, chosen, self.experts, self.top)
         inner = ops.moe_gate_up(h, self.w_gate_up, routing, out_dtype=ctx.dtype, limit=self.limit, alpha=self.alpha,
                                 shift=self.shift)                                     # [T * top, inner]
@@ -187,6 +192,15 @@ class RoutedExperts(FeedForward):
         import torch
         zero = torch.zeros((h.shape[0], self.width), dtype=torch.float32, device=h.device)
         return [(self.forward(ctx, h, zero), 1.0)]
+
+    def row_branches(self, ctx, h):
+        """The chosen experts' rows with their weights as factors, so that the caller's sum is the experts' too."""
+        import torch
+        if self.shared is not None:
+            return self.branches(ctx, h)
+        logits = ctx.ops.linear(h, self.w_router, None, out_dtype=torch.float32)
+        y, weights = self._chosen(ctx, h, logits)
+        return [(y[:, k, :], weights[:, k]) for k in range(self.top)]
 
 
 register_part("ffn", "routed_experts", RoutedExperts)

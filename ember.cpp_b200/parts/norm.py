@@ -57,6 +57,21 @@ class RMSNorm(Norm):
         """One launch: the weighted sum of the branches, its norm, and the sum with the stream."""
         return ctx.ops.add_normed(x, plain_branches(ctx, branches), self.w, self.eps, offset=self.offset)
 
+    def sum_normed(self, ctx, x, alpha, branches, average=None):
+        """One launch: the weighted sum of the stream and the branches (those with norms of their own included), its norm,
+        the sum over depth where one follows, and the rows in the compute type for the products that come next."""
+        eps = {b[2][1] for b in branches if len(b) > 2 and b[2] is not None}
+        if len(eps) > 1:        # (one launch takes one eps: norms of different eps are carried out first)
+            branches, eps = plain_branches(ctx, branches), set()
+        flat = [(b[0], b[1], b[2][0] if len(b) > 2 and b[2] is not None else None) for b in branches]
+        history, weights = (None, None) if average is None else average.fold(ctx)
+        y, stream, rows = ctx.ops.post_norm(x, alpha, flat, self.w, self.eps, self.offset, ctx.dtype,
+                                            branch_eps=eps.pop() if eps else 0.0, history=history, coef=weights)
+        if average is not None:
+            average.keep(ctx, y)
+        ctx.note_rows(stream, rows)
+        return stream
+
 
 class LayerScale(Norm):
     """A gain per channel and nothing else: `x * w`.  In the place of a norm after a sublayer (the `sandwich`

@@ -14,7 +14,9 @@ of pair i is a blend of f_i / factor and f_i by a ramp over the pair index, the 
 the indices whose wavelengths make `fast` and `slow` turns within the `original` context, and both
 cos and sin are multiplied by 0.1 ln(factor) + 1.  Frequencies are computed once on the host, the
 angles and their cos and sin in float32 on the device.  With `interleaved` the pairs are neighbours:
-dimension 2i with dimension 2i + 1.  A mixer that rotates only a part of its heads, or with constants
+dimension 2i with dimension 2i + 1.  `scaling` with `kind` "bands" (Llama 3.1's) scales by wavelength instead: a frequency
+whose wavelength 2 pi / f is below original / high stays, one above original / low becomes f / factor, and between the two
+it is (1 - s) f / factor + s f with s = (original / wavelength - low) / (high - low); cos and sin are not multiplied.  A mixer that rotates only a part of its heads, or with constants
 of its own, builds one of these for itself and calls `rotate`.
 """
 from __future__ import annotations
@@ -62,7 +64,18 @@ class Rotary(Position):
         half = self.dims // 2
         freqs = [self.base ** (-2.0 * i / self.dims) for i in range(half)]
         self.magnitude = 1.0
-        if scaling:
+        if scaling and scaling.get("kind", "yarn") not in ("yarn", "bands"):
+            raise ValueError(f"rotary {prefix!r}: scaling of kind {scaling['kind']!r}")
+        if scaling and scaling.get("kind") == "bands":
+            factor, original, low, high = (float(scaling[k]) for k in ("factor", "original", "low", "high"))
+            for i, f in enumerate(freqs):
+                wave = 2 * math.pi / f
+                if wave > original / low:
+                    freqs[i] = f / factor
+                elif wave >= original / high:
+                    s = (original / wave - low) / (high - low)
+                    freqs[i] = (1.0 - s) * f / factor + s * f
+        elif scaling:
             factor, original = float(scaling["factor"]), float(scaling["original"])
 
             def pair_at(turns):      # the pair index whose wavelength makes `turns` turns within the original context

@@ -38,6 +38,7 @@ class LayerSpec:
     ffn: PartSpec | None
     more_norms: tuple[tuple[str, PartSpec], ...] = ()
     addons: tuple[PartSpec, ...] = ()
+    block_params: dict[str, Any] = dataclasses.field(default_factory=dict)    # the arrangement's own constants
 
 
 @dataclasses.dataclass(frozen=True)

@@ -206,6 +206,78 @@ class CpuOps:
         z = proj[:, z_col:z_col + a.shape[1]].float()
         return (a.float() * (torch.sigmoid(z) if gate == "sigmoid" else z * torch.sigmoid(z))).to(a.dtype)
 
+    # ------------------------------------------------------------------ norms after the sum, sums over depth
+    def cast_rows(self, x, dtype):
+        return x.to(dtype)
+
+    def depth_average(self, history, coef, dtype):
+        stream = sum(c * t for c, t in zip(coef, history))
+        return stream, stream.to(dtype)
+
+    def post_norm(self, x, alpha, branches, w, eps, offset, dtype, branch_eps=0.0, history=None, coef=None):
+        total = alpha * x
+        for b in branches:
+            rows, f = b[0].float(), b[1]
+            if len(b) > 2 and b[2] is not None:
+                rows = rows * torch.rsqrt((rows * rows).mean(-1, keepdim=True) + branch_eps) * b[2]
+            total = total + rows * (f[:, None] if torch.is_tensor(f) else f)
+        y = self.rmsnorm(total, w, eps, torch.float32, offset)
+        stream = y if history is None else self.depth_average(list(history) + [y], coef, torch.float32)[0]
+        return y, stream, stream.to(dtype)
+
+    def qkv_prepare(self, proj, plan, cache, heads, kv_heads, head_dim, value_dim, out_dtype, store, v_col=None, norm=None,
+                    q_gain=None, k_gain=None, eps=0.0, rotary=None, unit_after=False):
+        T, q_w, k_w = plan.T, heads * head_dim, kv_heads * head_dim
+        unit = lambda t: t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps)  # noqa: E731
+
+        def heads_of(col, count, gain):
+            x = proj[:, col:col + count * head_dim].float()
+            if norm == "row":
+                x = unit(x) * (1.0 if gain is None else gain)
+            x = x.reshape(T, count, head_dim)
+            if norm == "head":
+                x = unit(x) * (1.0 if gain is None else gain)
+            x = x.reshape(T, count * head_dim).contiguous()
+            if rotary is not None:
+                self.rotate(x, x, plan.positions, count, 0, head_dim, 0, head_dim, head_dim, rotary.freqs, rotary.magnitude,
+                            rotary.dims, interleaved=rotary.interleaved)
+            if unit_after:
+                x = unit(x.reshape(T, count, head_dim)).reshape(T, count * head_dim)
+            return x
+        out = torch.full((T, q_w + k_w + kv_heads * value_dim), float("nan"))
+        out[:, :q_w] = heads_of(0, heads, q_gain)
+        if store:
+            v0 = q_w + k_w if v_col is None else v_col
+            rows = torch.cat([out[:, :q_w], heads_of(q_w, kv_heads, k_gain), proj[:, v0:v0 + kv_heads * value_dim].float()], 1)
+            self.kv_store(rows, cache, plan, heads, kv_heads, head_dim, value_dim)
+        return out.to(out_dtype)
+
+    def poly_norm(self, z, four, eps, out_dtype):
+        z = z.float()
+        unit = lambda t: t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps)  # noqa: E731
+        return (four[0] * unit(z) + four[1] * unit(z ** 2) + four[2] * unit(z ** 3) + four[3]).to(out_dtype)
+
+    def rglru(self, u, proj, y_col, w_gates, bias_r, bias_i, rate, state, plan):
+        T, width = u.shape
+        parts, _, n = w_gates.shape
+        z = torch.einsum("tbi,boi->tbo", u.float().view(T, parts, n), w_gates.float())
+        r = torch.sigmoid(z[:, :, :n].reshape(T, width) + bias_r)
+        i = torch.sigmoid(z[:, :, n:].reshape(T, width) + bias_i)
+        log_a = -rate * r
+        a, b = torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * i * u.float()
+        y = proj[:, y_col:y_col + width].float()
+        y = 0.5 * y * (1 + torch.tanh(math.sqrt(2 / math.pi) * (y + 0.044715 * y ** 3)))
+        out = torch.zeros(T, width)
+        for slot, start, t0, t1 in self._sequences(plan):
+            if slot < 0:
+                continue
+            S = state[slot].clone() if start > 0 else torch.zeros(width)
+            for t in range(t0, t1):
+                S = a[t] * S + b[t]
+                out[t] = S * y[t]
+            state[slot] = S
+        return out.to(u.dtype)
+
     # ------------------------------------------------------------------ mLSTM, minGRU
     def mlstm_gates(self, h, w, bias, heads, cap):
         g = h.float() @ w.float().t() + bias
@@ -359,7 +431,10 @@ class CpuOps:
             return table[:T].long()
         return table[tokens[:T].long()].long()            # [T, top]: the expert of every (token, choice) pair
 
-    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale):
+    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale, softmax=False):
+        if softmax:
+            picked, chosen = (logits[:, :experts].float() + correction).topk(top, dim=-1)
+            return chosen.to(torch.int32), torch.softmax(picked, -1) * route_scale
         s = torch.sigmoid(logits[:, :experts].float())
         choice = s + correction
         per = experts // groups
