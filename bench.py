@@ -247,6 +247,41 @@ VIPOLIX_SIZES = {
 }
 
 
+MAMUSUN_SIZES = {
+    # the recurrence's width / its blocks / taps of its convolution; rotated dimensions of the attention beside it
+    "small": dict(lru=1280, blocks=10, conv=4, rot=32),
+    "medium": dict(lru=2560, blocks=10, conv=4, rot=64),
+}
+
+
+def mamusun_config(size: str):
+    """A Mamusun of the width, layer count, attention heads, window, inner sizes, experts and vocabulary of
+    `DESIGN_SIZES[size]`: attention beside the recurrence with experts, an attention over all keys whose values are its keys
+    with a dense feed-forward, a windowed attention with experts, and one that reads its keys and values with a dense
+    feed-forward, in turn."""
+    z, m = DESIGN_SIZES[size], MAMUSUN_SIZES[size]
+    heads = {"dim": z["dim"], "vdim": z["dim"], "heads": z["heads"], "kv_heads": z["kv_heads"], "scale": z["dim"] ** -0.5}
+    window = {"mask": {"size": z["window"]}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"]}}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    bands = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}
+    yarn = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    layers = []
+    for i in range(z["layers"]):
+        if i % 4 == 0:
+            left = {**heads, **window, "rot": {"dims": m["rot"], "base": 500000.0, "scaling": bands}}
+            right = {"width": m["lru"], "blocks": m["blocks"], "conv": m["conv"]}
+            layers.append({"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": dict(moe)})
+        elif i % 4 == 1:
+            rot = {"dims": z["dim"], "base": 500000.0, "scaling": yarn}
+            layers.append({"type": "attention_2", "mixer": {**heads, "rot": rot}, "mlp": dict(dense)})
+        else:
+            more = {} if i % 4 == 2 else {"kv_from": i - 1}
+            layers.append({"type": "attention", "mixer": {**heads, **window, **more}, "mlp": dict(moe if i % 4 == 2 else dense)})
+    return {"architecture": "Mamusun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "postln_alpha": 1.5,
+            "layers": layers}
+
+
 def vipolix_config(size: str):
     """A Vipolix of the width, layer count, attention heads, chunk (the others' window), experts and vocabulary of
     `DESIGN_SIZES[size]`: layers of gated linear attention and of attention beside the generalized delta rule in turn, every
@@ -314,6 +349,8 @@ def design_configs(size: str, design: str = "nipolorn"):
         return (muzozen_config(size),) + design_configs(size)
     if design == "sosutar":
         return (sosutar_config(size),) + design_configs(size)
+    if design == "mamusun":
+        return (mamusun_config(size),) + design_configs(size)
     if design == "vipolix":
         return (vipolix_config(size),) + design_configs(size)
     z = DESIGN_SIZES[size]
@@ -449,7 +486,7 @@ def main() -> int:
                     help="time one bfloat16 product on every kernel that takes it, instead of the benchmark")
     ap.add_argument("--act", default=None, choices=[None, "gelu_tanh", "gelu_erf"], help="with --linear: the epilogue's activation")
     ap.add_argument("--residual", action="store_true", help="with --linear: add a float32 residual (the output is float32 then)")
-    ap.add_argument("--design", default=None, choices=["nipolorn", "muzozen", "sosutar", "vipolix"],
+    ap.add_argument("--design", default=None, choices=["nipolorn", "muzozen", "sosutar", "vipolix", "mamusun"],
                     help="instead of the benchmark: prefill and decode throughput of this design beside a GPT-2 of equal size "
                          "(muzozen: beside a Nipolorn and a GPT-2 of equal size)")
     ap.add_argument("--design-size", default="medium", choices=sorted(DESIGN_SIZES), help="with --design: the layers' sizes")

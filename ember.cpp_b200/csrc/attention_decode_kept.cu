@@ -7,7 +7,8 @@
 // In a block each of four warps takes 32 keys, a key a lane: the lane reads its key's row in 16-byte pieces
 // and makes the dot products with every query head of the group (the queries lie in shared memory, read by
 // all lanes at once); one maximum and one correction per head for the warp's 32 keys; then the 32 value rows
-// are walked through together, every lane owning a run of the value dims.  Softmax, sums and accumulators are
+// are walked through together, every lane owning a run of the value dims.  Both walks ask for several rows' pieces before
+// they use the first, so that a block waits for memory a few times and not once a key.  Softmax, sums and accumulators are
 // float32.  Partial results (m, l, acc[vd]) per (token, head, chunk) go to scratch that the caller gives.
 // With `slopes` the score of key j loses slopes[head] * (p - j); with `sinks` the merge adds exp(sinks[head]) to the
 // softmax's denominator (a term without a key or a value).
@@ -27,7 +28,7 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
                            const int* __restrict__ pages, int max_blocks, int n_heads, int kv_heads, int hd, int vd,
                            float scale, int window, int keep_first, int n_chunks, const float* __restrict__ slopes, int chunk,
                            const float* __restrict__ head_scales) {
-  __shared__ float q_s[PER][256];
+  __shared__ __align__(16) float q_s[PER][256];
   __shared__ float m_s[kWarps][PER], l_s[kWarps][PER];
   __shared__ float acc_s[kWarps][PER][32 * DPL];
   const int c = blockIdx.x, g = blockIdx.y, t = blockIdx.z;
@@ -67,21 +68,31 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
   for (int h = 0; h < PER; ++h) sc[h] = 0.f;
   if (valid) {
     const __nv_bfloat16* k = kc + row * hd;
-    for (int d = 0; d < hd; d += 8) {  // (head sizes are multiples of 8: rows of 16-byte pieces)
-      const uint4 raw = *reinterpret_cast<const uint4*>(k + d);
-      const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
-      float kv[8];
+    constexpr int kPieces = 8;
+    for (int d0 = 0; d0 < hd; d0 += 8 * kPieces) {  // (head sizes are multiples of 8: rows of 16-byte pieces)
+      uint4 raw[kPieces];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float2 f = __bfloat1622float2(h2[i]);
-        kv[2 * i] = f.x;
-        kv[2 * i + 1] = f.y;
-      }
+      for (int u = 0; u < kPieces; ++u)
+        raw[u] = d0 + 8 * u < hd ? *reinterpret_cast<const uint4*>(k + d0 + 8 * u) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
-      for (int h = 0; h < PER; ++h) {
-        if (h < per) {
+      for (int u = 0; u < kPieces; ++u) {
+        const int d = d0 + 8 * u;
+        if (d >= hd) break;
+        const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
+        float kv[8];
 #pragma unroll
-          for (int i = 0; i < 8; ++i) sc[h] = fmaf(q_s[h][d + i], kv[i], sc[h]);
+        for (int i = 0; i < 4; ++i) {
+          const float2 f = __bfloat1622float2(h2[i]);
+          kv[2 * i] = f.x;
+          kv[2 * i + 1] = f.y;
+        }
+#pragma unroll
+        for (int h = 0; h < PER; ++h) {
+          if (h < per) {
+            const float4 qa = *reinterpret_cast<const float4*>(&q_s[h][d]), qb = *reinterpret_cast<const float4*>(&q_s[h][d + 4]);
+            sc[h] = fmaf(qa.x, kv[0], fmaf(qa.y, kv[1], fmaf(qa.z, kv[2], fmaf(qa.w, kv[3], sc[h]))));
+            sc[h] = fmaf(qb.x, kv[4], fmaf(qb.y, kv[5], fmaf(qb.z, kv[6], fmaf(qb.w, kv[7], sc[h]))));
+          }
         }
       }
     }
@@ -107,32 +118,39 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
     for (int i = 0; i < DPL; ++i) acc[h][i] = 0.f;
   const int n_valid = min(32, k1 - (k0 + warp * 32));  // <= 0: this warp has no keys
   const bool dims = lane * DPL < vd;
-  for (int jj = 0; jj < n_valid; ++jj) {
-    const unsigned long long r = __shfl_sync(0xffffffffu, (unsigned long long)row, jj);
-    const int there = __shfl_sync(0xffffffffu, (int)valid, jj);
-    float v[DPL];
+  constexpr int kRowsAhead = 8;
+  for (int j0 = 0; j0 < n_valid; j0 += kRowsAhead) {
+    unsigned raw[kRowsAhead][DPL == 4 ? 2 : 1];     // a lane's values of a row: DPL of two bytes
 #pragma unroll
-    for (int i = 0; i < DPL; ++i) v[i] = 0.f;
-    if (dims && there) {
-      const __nv_bfloat16* vr = vc + r * vd + lane * DPL;
-      if constexpr (DPL == 4) {
-        const uint2 raw = *reinterpret_cast<const uint2*>(vr);
-        const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
-        const float2 a = __bfloat1622float2(h2[0]), b = __bfloat1622float2(h2[1]);
-        v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
-      } else if constexpr (DPL == 2) {
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vr));
-        v[0] = a.x, v[1] = a.y;
-      } else {
-#pragma unroll
-        for (int i = 0; i < DPL; ++i) v[i] = __bfloat162float(vr[i]);
+    for (int u = 0; u < kRowsAhead; ++u) {           // (a lane without a key has probability zero and no row)
+      const unsigned long long r = __shfl_sync(0xffffffffu, (unsigned long long)row, j0 + u);
+      const int there = __shfl_sync(0xffffffffu, (int)valid, j0 + u);
+      raw[u][0] = 0u;
+      if constexpr (DPL == 4) raw[u][1] = 0u;
+      if (dims && there) {
+        const __nv_bfloat16* vr = vc + r * vd + lane * DPL;
+        if constexpr (DPL == 4) {
+          const uint2 two = *reinterpret_cast<const uint2*>(vr);
+          raw[u][0] = two.x, raw[u][1] = two.y;
+        } else if constexpr (DPL == 2) {
+          raw[u][0] = *reinterpret_cast<const unsigned*>(vr);
+        } else {
+          raw[u][0] = *reinterpret_cast<const unsigned short*>(vr);
+        }
       }
     }
 #pragma unroll
-    for (int h = 0; h < PER; ++h) {
-      const float pv = __shfl_sync(0xffffffffu, pj[h], jj);
+    for (int u = 0; u < kRowsAhead; ++u) {
+      float v[DPL];
 #pragma unroll
-      for (int i = 0; i < DPL; ++i) acc[h][i] = fmaf(pv, v[i], acc[h][i]);
+      for (int i = 0; i < DPL; ++i)      // bfloat16 is the upper half of a float
+        v[i] = __uint_as_float(i % 2 == 0 ? raw[u][i / 2] << 16 : raw[u][i / 2] & 0xffff0000u);
+#pragma unroll
+      for (int h = 0; h < PER; ++h) {
+        const float pv = __shfl_sync(0xffffffffu, pj[h], j0 + u);
+#pragma unroll
+        for (int i = 0; i < DPL; ++i) acc[h][i] = fmaf(pv, v[i], acc[h][i]);
+      }
     }
   }
   if (n_valid <= 0 && lane == 0) {
@@ -181,21 +199,37 @@ __global__ void decode_kept_merge_kernel(const float* __restrict__ part, __nv_bf
   }
   const size_t stride = (size_t)vd + 2;
   const float* src = part + (size_t)item * n_chunks * stride;
+  const int lane = threadIdx.x & 31;
+  // every warp for itself: a lane a chunk (32 at a time) for the maximum, then for the factors e^(m_c - M) and the sum
   float m = sinks ? sinks[item % n_heads] : -INFINITY;
-  for (int c = 0; c < n_chunks; ++c) m = fmaxf(m, src[c * stride]);
+  for (int c0 = 0; c0 < n_chunks; c0 += 32) m = fmaxf(m, warp_max(c0 + lane < n_chunks ? src[(c0 + lane) * stride] : -INFINITY));
   float l = sinks ? expf(sinks[item % n_heads] - m) : 0.f;
-  for (int c = 0; c < n_chunks; ++c) {
-    const float mc = src[c * stride];
-    if (mc != -INFINITY) l = fmaf(src[c * stride + 1], expf(mc - m), l);
+  constexpr int kDims = 1;               // value dims a thread (the launch has a thread a dim)
+  float a[kDims];
+#pragma unroll
+  for (int e = 0; e < kDims; ++e) a[e] = 0.f;
+  for (int c0 = 0; c0 < n_chunks; c0 += 32) {
+    const bool mine = c0 + lane < n_chunks;
+    const float mc = mine ? src[(c0 + lane) * stride] : -INFINITY;
+    const float f = mc == -INFINITY ? 0.f : expf(mc - m);
+    l += warp_sum(f == 0.f ? 0.f : src[(c0 + lane) * stride + 1] * f);
+    const int count = min(32, n_chunks - c0);
+#pragma unroll 4
+    for (int c = 0; c < count; ++c) {
+      const float fc = __shfl_sync(0xffffffffu, f, c);
+      if (fc == 0.f) continue;           // (a chunk without keys left nothing there; the same for every lane)
+#pragma unroll
+      for (int e = 0; e < kDims; ++e) {
+        const int d = threadIdx.x + e * blockDim.x;
+        if (d < vd) a[e] = fmaf(src[(c0 + c) * stride + 2 + d], fc, a[e]);
+      }
+    }
   }
   const float inv = 1.0f / l;
-  for (int d = threadIdx.x; d < vd; d += blockDim.x) {
-    float a = 0.f;
-    for (int c = 0; c < n_chunks; ++c) {
-      const float mc = src[c * stride];
-      if (mc != -INFINITY) a = fmaf(src[c * stride + 2 + d], expf(mc - m), a);
-    }
-    o[d] = __float2bfloat16_rn(a * inv);
+#pragma unroll
+  for (int e = 0; e < kDims; ++e) {
+    const int d = threadIdx.x + e * blockDim.x;
+    if (d < vd) o[d] = __float2bfloat16_rn(a[e] * inv);
   }
 }
 

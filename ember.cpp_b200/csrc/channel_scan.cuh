@@ -8,11 +8,12 @@
 // slot's state holds; sequences of slot -1 are padding: their rows are zero and no state is touched.
 //
 // A rule has
-//   struct Row            the values of one token and channel, as fetched
-//   begin(c)              what a channel keeps (biases)
-//   fetch(t, c, with_out) a token's Row (with_out false: what only the result needs may be left out)
-//   factors(row, A, B)    A_t and B_t
-//   result(row, S)        the token's output
+//   struct Row               the values of one token and channel, as fetched
+//   begin(c)                 what a channel keeps (biases)
+//   fetch(t, c, phase)       a token's Row for a phase (see the kernel: what a phase does not need may be left out)
+//   factors(row, phase, A, B)  A_t and B_t
+//   keep(t, c, A, B)         the first walk's factors, for a rule that leaves them to the second walk (or nothing)
+//   result(row, S)           the token's output
 #pragma once
 
 #include "common.cuh"
@@ -24,10 +25,10 @@ constexpr int kThreads = 128;
 // grid (sequences, channel tiles, pieces).  phase 0: the whole walk (one piece).  phase 1: a piece from zero,
 // leaving (product of A, end value) in scratch.  phase 2: the walk from the piece's start value, which the
 // carry left in scratch.
-template <typename Rule, typename TOUT>
+template <int phase, typename Rule, typename TOUT>
 __global__ void __launch_bounds__(kThreads)
 channel_scan_kernel(Rule rule, float* __restrict__ state, TOUT* __restrict__ out, const int* __restrict__ seq_slot,
-                    const int* __restrict__ seq_start, const int* __restrict__ cu_new, int width, int piece, int phase,
+                    const int* __restrict__ seq_start, const int* __restrict__ cu_new, int width, int piece,
                     float* __restrict__ scratch) {
   const int s = blockIdx.x, c = blockIdx.y * kThreads + threadIdx.x, p = blockIdx.z;
   if (c >= width) return;
@@ -46,19 +47,36 @@ channel_scan_kernel(Rule rule, float* __restrict__ state, TOUT* __restrict__ out
   if (phase == 0) S = seq_start[s] > 0 ? state[(size_t)slot * width + c] : 0.f;
   if (phase == 2) S = mine[1];
   float all = 1.f;
-  constexpr int kAhead = 8;      // tokens whose columns are fetched before the chain of the state walks them
-  for (int i0 = lo; i0 < hi; i0 += kAhead) {
+  constexpr int kAhead = 8;      // tokens whose columns are fetched, and whose factors are made, before the chain walks them
+  int i0 = lo;
+  for (; i0 + kAhead <= hi; i0 += kAhead) {
     typename Rule::Row rows[kAhead];
+    float A[kAhead], B[kAhead];
 #pragma unroll
-    for (int u = 0; u < kAhead; ++u) rows[u] = rule.fetch((size_t)(t0 + (i0 + u < hi ? i0 + u : lo)), c, phase != 1);
+    for (int u = 0; u < kAhead; ++u) rows[u] = rule.fetch((size_t)(t0 + i0 + u), c, phase);
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) rule.factors(rows[u], phase, A[u], B[u]);
 #pragma unroll
     for (int u = 0; u < kAhead; ++u) {
-      if (i0 + u >= hi) break;
-      float A, B;
-      rule.factors(rows[u], A, B);
-      S = fmaf(A, S, B);
-      if (phase == 1) all *= A;
-      else out[(size_t)(t0 + i0 + u) * width + c] = from_float<TOUT>(rule.result(rows[u], S));
+      S = fmaf(A[u], S, B[u]);
+      if (phase == 1) {
+        all *= A[u];
+        rule.keep((size_t)(t0 + i0 + u), c, A[u], B[u]);
+      } else {
+        out[(size_t)(t0 + i0 + u) * width + c] = from_float<TOUT>(rule.result(rows[u], S));
+      }
+    }
+  }
+  for (; i0 < hi; ++i0) {
+    float A, B;
+    const typename Rule::Row row = rule.fetch((size_t)(t0 + i0), c, phase);
+    rule.factors(row, phase, A, B);
+    S = fmaf(A, S, B);
+    if (phase == 1) {
+      all *= A;
+      rule.keep((size_t)(t0 + i0), c, A, B);
+    } else {
+      out[(size_t)(t0 + i0) * width + c] = from_float<TOUT>(rule.result(row, S));
     }
   }
   if (phase == 1) {
@@ -94,16 +112,16 @@ template <typename Rule, typename TOUT>
 cudaError_t launch(const Rule& rule, float* state, TOUT* out, const int* seq_slot, const int* seq_start, const int* cu_new,
                    int n_seqs, int width, int piece, int pieces, float* scratch, cudaStream_t stream) {
   const int tiles = (width + kThreads - 1) / kThreads;
-  auto walk = [&](int phase, int count) {
-    return launch_plain(channel_scan_kernel<Rule, TOUT>, dim3(n_seqs, tiles, count), dim3(kThreads), 0, stream, rule, state, out,
-                        seq_slot, seq_start, cu_new, width, piece, phase, scratch);
+  auto walk = [&](auto kernel, int count) {
+    return launch_plain(kernel, dim3(n_seqs, tiles, count), dim3(kThreads), 0, stream, rule, state, out, seq_slot, seq_start, cu_new,
+                        width, piece, scratch);
   };
-  if (pieces == 1) return walk(0, 1);
-  cudaError_t e = walk(1, pieces);
+  if (pieces == 1) return walk(channel_scan_kernel<0, Rule, TOUT>, 1);
+  cudaError_t e = walk(channel_scan_kernel<1, Rule, TOUT>, pieces);
   if (e == cudaSuccess)
     e = launch_plain(channel_carry_kernel, dim3(n_seqs, tiles), dim3(kThreads), 0, stream, scratch, (const float*)state, seq_slot,
                      seq_start, cu_new, width, piece, pieces);
-  return e == cudaSuccess ? walk(2, pieces) : e;
+  return e == cudaSuccess ? walk(channel_scan_kernel<2, Rule, TOUT>, pieces) : e;
 }
 
 }  // namespace scan

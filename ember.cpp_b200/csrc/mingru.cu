@@ -24,11 +24,12 @@ struct MinGru {
     bz = bias_z[c];
     bx = bias_x[c];
   }
-  __device__ __forceinline__ Row fetch(size_t t, int c, bool with_out) const {
+  __device__ __forceinline__ Row fetch(size_t t, int c, int phase) const {
     const TIN* row = proj + t * stride;
-    return Row{to_float(row[z_col + c]), to_float(row[x_col + c]), with_out ? to_float(row[g_col + c]) : 0.f};
+    return Row{to_float(row[z_col + c]), to_float(row[x_col + c]), phase != 1 ? to_float(row[g_col + c]) : 0.f};
   }
-  __device__ __forceinline__ void factors(const Row& r, float& A, float& B) const {
+  __device__ __forceinline__ void keep(size_t, int, float, float) const {}
+  __device__ __forceinline__ void factors(const Row& r, int, float& A, float& B) const {
     const float z = sigmoidf(r.z + bz), b = r.x + bx;
     A = 1.0f - z;
     B = z * (b >= 0.f ? b + 0.5f : sigmoidf(b));

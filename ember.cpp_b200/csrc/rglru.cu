@@ -5,26 +5,30 @@
 //     S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t                         out_t = S_t * gelu_tanh(y_t)
 // rate >= 0 is a constant of the channel (a factor times softplus of a learned number).  zr and zi are products of u with
 // a square matrix for each of `parts` equal parts of the channels: rows of 2 * width values in which part b holds its
-// n = width / parts values of zr, then its n values of zi.  Everything from the products on is float32.
+// n = width / parts values of zr, then its n values of zi.  Everything from the products on is float32.  With
+// m = exp(log a) - 1 (one expm1), a = 1 + m and 1 - a^2 = -m (2 + m), exact where a is close to one.
 //
-//   ember_rglru       the recurrence over rows of zr | zi (the walk is channel_scan.cuh's)
+//   ember_rglru       the recurrence over rows of zr | zi (the walk is channel_scan.cuh's; where pieces are walked twice, the
+//                     first walk leaves a and sqrt(1 - a^2) i u in the places of zr and zi for the second)
 //   ember_rglru_step  steps that bring one token a sequence: the products of the gates and the recurrence in one launch;
 //                     a warp makes both gates of a channel for eight sequences, so that a matrix row is read once for them
 #include "channel_scan.cuh"
 
 namespace {
 
-__device__ __forceinline__ float sigmoidf(float v) { return 1.0f / (1.0f + expf(-v)); }
+__device__ __forceinline__ float sigmoidf(float v) { return __fdividef(1.0f, 1.0f + expf(-v)); }
+// the tanh form of GELU, 0.5 (1 + tanh(x)) being sigmoid(2 x)
+__device__ __forceinline__ float gelu_gate(float v) { return v * sigmoidf(1.5957691216057308f * (v + 0.044715f * v * v * v)); }
 
 __device__ __forceinline__ void rglru_factors(float zr, float zi, float u, float rate, float& A, float& B) {
-  const float log_a = -rate * sigmoidf(zr);
-  A = expf(log_a);
-  B = sqrtf(fmaxf(-expm1f(2.0f * log_a), 0.f)) * sigmoidf(zi) * u;
+  const float m = expm1f(-rate * sigmoidf(zr));
+  A = 1.0f + m;
+  B = sqrtf(-m * (2.0f + m)) * sigmoidf(zi) * u;      // (-1 <= m <= 0)
 }
 
 template <typename T>
 struct RgLru {
-  const float* gates;       // [T, 2 * width]
+  float* gates;             // [T, 2 * width]
   const T* u;               // [T, width]
   const T* y;               // rows of y_stride values, the channel's value at column c
   long long y_stride;
@@ -41,14 +45,20 @@ struct RgLru {
     rt = rate[c];
     col = c / part * 2 * part + c % part;
   }
-  __device__ __forceinline__ Row fetch(size_t t, int c, bool with_out) const {
+  __device__ __forceinline__ Row fetch(size_t t, int c, int phase) const {
     const float* g = gates + t * 2 * width + col;
-    return Row{g[0], g[part], to_float(u[t * width + c]), with_out ? to_float(y[t * y_stride + c]) : 0.f};
+    return Row{g[0], g[part], phase != 2 ? to_float(u[t * width + c]) : 0.f, phase != 1 ? to_float(y[t * y_stride + c]) : 0.f};
   }
-  __device__ __forceinline__ void factors(const Row& r, float& A, float& B) const {
-    rglru_factors(r.zr + br, r.zi + bi, r.u, rt, A, B);
+  __device__ __forceinline__ void factors(const Row& r, int phase, float& A, float& B) const {
+    if (phase == 2) A = r.zr, B = r.zi;
+    else rglru_factors(r.zr + br, r.zi + bi, r.u, rt, A, B);
   }
-  __device__ __forceinline__ float result(const Row& r, float S) const { return S * gelu_tanh(r.y); }
+  __device__ __forceinline__ void keep(size_t t, int, float A, float B) const {
+    float* g = gates + t * 2 * width + col;
+    g[0] = A;
+    g[part] = B;
+  }
+  __device__ __forceinline__ float result(const Row& r, float S) const { return S * gelu_gate(r.y); }
 };
 
 constexpr int kStepWarps = 8;
@@ -104,16 +114,16 @@ rglru_step_kernel(const __nv_bfloat16* __restrict__ u, const __nv_bfloat16* __re
   float* st = state + (size_t)slot * width + ch;
   const float S = fmaf(A, seq_start[t] > 0 ? *st : 0.f, B);
   *st = S;
-  *o = __float2bfloat16_rn(S * gelu_tanh(__bfloat162float(y[(size_t)t * y_stride + ch])));
+  *o = __float2bfloat16_rn(S * gelu_gate(__bfloat162float(y[(size_t)t * y_stride + ch])));
 }
 
 }  // namespace
 
 EMBER_API size_t ember_rglru_scratch(int n_seqs, int pieces, int width) { return scan::scratch_floats(n_seqs, pieces, width); }
 
-// gates float32 [T, 2 * width] (see above), u [T, width] and y (rows of y_stride values) of one element type, biases and
+// gates float32 [T, 2 * width] (see above; overwritten where pieces > 1), u [T, width] and y (rows of y_stride values) of one element type, biases and
 // rate float32 [width], state float32 [slots, width] (advanced), out [T, width] of u's type.
-EMBER_API int ember_rglru(const float* gates, const void* u, const void* y, long long y_stride, const float* bias_r,
+EMBER_API int ember_rglru(float* gates, const void* u, const void* y, long long y_stride, const float* bias_r,
                           const float* bias_i, const float* rate, float* state, void* out, const int* seq_slot,
                           const int* seq_start, const int* cu_new, int n_seqs, int width, int parts, int piece, int pieces,
                           float* scratch, int dtype, cudaStream_t stream) {

@@ -158,6 +158,86 @@ post_norm_kernel(const float* __restrict__ x, float alpha, const Branches b, con
   }
 }
 
+// The same for rows of up to 4 x blockDim.x values and NB branches or fewer: every thread has four values of each tensor
+// in registers and asks for all of them before the first sum, so that a launch of few rows waits for memory once.
+template <int NB>
+__global__ void __launch_bounds__(1024)
+post_norm_short_kernel(const float* __restrict__ x, float alpha, const Branches b, const float* __restrict__ w, float offset,
+                       float eps, float branch_eps, float* __restrict__ out, __nv_bfloat16* __restrict__ copy, const History hist,
+                       const float* __restrict__ coef, float* __restrict__ mean, int d) {
+  __shared__ float red[NB + 1][32];
+  const size_t row = blockIdx.x, base = row * (size_t)d;
+  const int i = threadIdx.x * 4, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const bool there = i < d;
+  const Vals<4> zero = {{0.f, 0.f, 0.f, 0.f}};
+  Vals<4> s = zero, g = zero, a = zero, v[NB], bg[NB];
+  float f[NB], c_last = 0.f;
+  bool normed = false;
+#pragma unroll
+  for (int k = 0; k < NB; ++k) {
+    v[k] = bg[k] = zero;
+    f[k] = 0.f;
+    if (k < b.n) {
+      if (there) v[k] = load_row<4>(b.rows[k] + row * (size_t)b.stride[k] + i);
+      if (there && b.gain[k]) bg[k] = load_row<4>(b.gain[k] + i);
+      f[k] = b.factor[k] * (b.weight[k] ? b.weight[k][row * (size_t)b.weight_stride[k]] : 1.f);
+      normed = normed || b.gain[k];
+    }
+  }
+  if (there) {
+    s = load_row<4>(x + base + i);
+    g = load_row<4>(w + i);
+    if (mean) {
+      a = history_sum<4>(hist, coef, base + i);
+      c_last = coef[hist.n];
+    }
+  }
+  if (normed) {        // (uniform over the block)
+#pragma unroll
+    for (int k = 0; k < NB; ++k) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss = fmaf(v[k].v[e], v[k].v[e], ss);
+      ss = warp_sum(ss);
+      if (lane == 0) red[k][warp] = ss;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < NB; ++k) {
+      if (k >= b.n || !b.gain[k]) continue;
+      float total = 0.f;
+      for (int q = 0; q < warps; ++q) total += red[k][q];
+      f[k] *= 1.0f / sqrtf(total / (float)d + branch_eps);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    float t = alpha * s.v[e];
+#pragma unroll
+    for (int k = 0; k < NB; ++k)
+      if (k < b.n) t = fmaf(b.gain[k] ? f[k] * bg[k].v[e] : f[k], v[k].v[e], t);
+    s.v[e] = t;
+    ss = fmaf(t, t, ss);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) red[NB][warp] = ss;
+  __syncthreads();
+  float total = 0.f;
+  for (int q = 0; q < warps; ++q) total += red[NB][q];
+  const float inv = 1.0f / sqrtf(total / (float)d + eps);
+  if (!there) return;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) s.v[e] = s.v[e] * inv * (offset + g.v[e]);
+  store_row<4>(out + base + i, s);
+  if (mean) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s.v[e] = fmaf(c_last, s.v[e], a.v[e]);
+    store_row<4>(mean + base + i, s);
+  }
+  if (copy) store_row<4>(copy + base + i, s);
+}
+
 template <int W>
 __global__ void __launch_bounds__(kThreads)
 depth_average_kernel(const History hist, const float* __restrict__ coef, float* __restrict__ mean, __nv_bfloat16* __restrict__ copy,
@@ -211,6 +291,18 @@ EMBER_API int ember_post_norm(const float* x, float alpha, const void* const* ro
   const int per = vec ? 4 : 1;
   const int threads = (d + per - 1) / per >= kThreads ? kThreads : ((d + per - 1) / per + 31) / 32 * 32;
   const size_t smem = (size_t)d * sizeof(float);
+  // (2,048 rows of 2,048: 26 microseconds a launch with the loop, 30 with the registers; 8 rows: 17 and 14.  Without a copy
+  // the stream is the compute type's own, float32: one kernel whatever the rows, so that every cut of the work adds alike)
+  if (vec && copy != nullptr && n_rows < 512 && d <= 4096 && n_branches <= 4) {
+    const int quads = (d / 4 + 31) / 32 * 32;
+#define EMBER_PN(NB)                                                                                                               \
+  launch_plain(post_norm_short_kernel<NB>, dim3(n_rows), dim3(quads), 0, stream, x, alpha, b, w, offset, eps, branch_eps, out, \
+               (__nv_bfloat16*)copy, h, coef, mean, d)
+    const cudaError_t e = n_branches == 1 ? EMBER_PN(1) : n_branches == 2 ? EMBER_PN(2) : EMBER_PN(4);
+#undef EMBER_PN
+    if (e != cudaSuccess) return ember_fail("post_norm: %s", cudaGetErrorString(e));
+    return 0;
+  }
   const cudaError_t e =
       vec ? launch_plain(post_norm_kernel<4>, dim3(n_rows), dim3(threads), smem, stream, x, alpha, b, w, offset, eps, branch_eps, out,
                          (__nv_bfloat16*)copy, h, coef, mean, d)

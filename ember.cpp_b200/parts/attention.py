@@ -246,16 +246,17 @@ class CausalAttention(Mixer):
                               q_gain=self.q_gain, k_gain=self.k_gain, eps=self.norm_eps, rotary=self.rotary, unit_after=self.unit_qk)
         more = dict(slopes=self.slopes, sinks=self.sinks, chunk=self.chunk, head_scales=self.head_scales,
                     head_scales_positive=self.head_scales is None or self.head_scales_positive)
-        if self._plain_sight(ctx.dtype):
+        if self._plain_sight():
             return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
                                  out_dtype=ctx.dtype, store=False)
         return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
                              out_dtype=ctx.dtype, store=False, keep_first=self.keep_first if self.window > 0 else 0,
                              value_dim=self.value_dim, **more)
 
-    def _plain_sight(self, dtype) -> bool:
-        """Nothing but a window on the scores, and sizes that the kernels for such heads have."""
-        return (not self.biased and self.keep_first == 0 and self.value_dim == self.head_dim and self.head_dim in (64, 128)
+    def _plain_sight(self) -> bool:
+        """Nothing but a window on the scores, and the head size at which the kernels for such heads are the faster ones (one
+        token each of 8 sequences at 2,048 positions, 16 heads over 4: 8.9 against 14.9 microseconds at 64, 25 against 19 at 128)."""
+        return (not self.biased and self.keep_first == 0 and self.value_dim == self.head_dim == 64
                 and self.n_heads // self.kv_heads <= 8 and self.scale > 0)
 
     def _attend(self, ctx, h, app):
