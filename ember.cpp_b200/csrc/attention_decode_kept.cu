@@ -4,9 +4,9 @@
 // of 128; a block takes one chunk of one key/value head of one token and serves all query heads of that
 // head, so that a key or value row is fetched once for the group; a second small launch merges the chunks.
 //
-// In a block each of four warps takes 32 keys, a key a lane: the lane reads its key's row in 16-byte pieces
-// and makes the dot products with every query head of the group (the queries lie in shared memory, read by
-// all lanes at once); one maximum and one correction per head for the warp's 32 keys; then the 32 value rows
+// In a block each of eight warps takes 16 keys, two lanes a key: a lane reads half of its key's row in 16-byte pieces
+// and makes that half of the dot products with every query head of the group (the queries lie in shared memory);
+// one maximum and one correction per head for the warp's 16 keys; then the 16 value rows
 // are walked through together, every lane owning a run of the value dims.  Both walks ask for several rows' pieces before
 // they use the first, so that a block waits for memory a few times and not once a key.  Softmax, sums and accumulators are
 // float32.  Partial results (m, l, acc[vd]) per (token, head, chunk) go to scratch that the caller gives.
@@ -16,8 +16,9 @@
 
 namespace {
 
-constexpr int kWarps = 4;
-constexpr int kChunkKeys = 32 * kWarps;
+constexpr int kWarps = 8;
+constexpr int kWarpKeys = 16;
+constexpr int kChunkKeys = kWarpKeys * kWarps;
 
 // PER: query heads a key/value head (rounded up); DPL: value dims a lane (vd <= 32 * DPL, vd % DPL == 0)
 template <int PER, int DPL>
@@ -57,7 +58,7 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
   __syncthreads();
 
   const int* my_pages = pages + (size_t)t * max_blocks;
-  const int idx = k0 + warp * 32 + lane;
+  const int idx = k0 + warp * kWarpKeys + (lane >> 1);
   const int j = idx < n_kept ? idx : lo + idx - n_kept;
   const int page = idx < k1 ? my_pages[j / kPage] : -1;
   const bool valid = page >= 0;
@@ -69,14 +70,15 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
   if (valid) {
     const __nv_bfloat16* k = kc + row * hd;
     constexpr int kPieces = 8;
-    for (int d0 = 0; d0 < hd; d0 += 8 * kPieces) {  // (head sizes are multiples of 8: rows of 16-byte pieces)
+    // (head sizes are multiples of 8: rows of 16-byte pieces, of which the key's two lanes take every other one)
+    for (int d0 = (lane & 1) * 8; d0 < hd; d0 += 16 * kPieces) {
       uint4 raw[kPieces];
 #pragma unroll
       for (int u = 0; u < kPieces; ++u)
-        raw[u] = d0 + 8 * u < hd ? *reinterpret_cast<const uint4*>(k + d0 + 8 * u) : make_uint4(0u, 0u, 0u, 0u);
+        raw[u] = d0 + 16 * u < hd ? *reinterpret_cast<const uint4*>(k + d0 + 16 * u) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
       for (int u = 0; u < kPieces; ++u) {
-        const int d = d0 + 8 * u;
+        const int d = d0 + 16 * u;
         if (d >= hd) break;
         const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
         float kv[8];
@@ -102,10 +104,11 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
   for (int h = 0; h < PER; ++h) {
     const float slope = slopes && h < per ? slopes[g * per + h] : 0.f;
     const float hs = head_scales && h < per ? scale * head_scales[g * per + h] : scale;
+    sc[h] += __shfl_xor_sync(0xffffffffu, sc[h], 1);
     const float s = valid ? sc[h] * hs - slope * (float)(p - j) : -INFINITY;
     const float m = warp_max(s);  // (the warp's first key is always there: m is finite)
     pj[h] = valid ? expf(s - m) : 0.f;
-    const float l = warp_sum(pj[h]);
+    const float l = 0.5f * warp_sum(pj[h]);     // (every key counts in two lanes)
     if (lane == 0) {
       m_s[warp][h] = m;
       l_s[warp][h] = l;
@@ -116,15 +119,15 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
   for (int h = 0; h < PER; ++h)
 #pragma unroll
     for (int i = 0; i < DPL; ++i) acc[h][i] = 0.f;
-  const int n_valid = min(32, k1 - (k0 + warp * 32));  // <= 0: this warp has no keys
+  const int n_valid = min(kWarpKeys, k1 - (k0 + warp * kWarpKeys));  // <= 0: this warp has no keys
   const bool dims = lane * DPL < vd;
   constexpr int kRowsAhead = 8;
   for (int j0 = 0; j0 < n_valid; j0 += kRowsAhead) {
     unsigned raw[kRowsAhead][DPL == 4 ? 2 : 1];     // a lane's values of a row: DPL of two bytes
 #pragma unroll
     for (int u = 0; u < kRowsAhead; ++u) {           // (a lane without a key has probability zero and no row)
-      const unsigned long long r = __shfl_sync(0xffffffffu, (unsigned long long)row, j0 + u);
-      const int there = __shfl_sync(0xffffffffu, (int)valid, j0 + u);
+      const unsigned long long r = __shfl_sync(0xffffffffu, (unsigned long long)row, 2 * (j0 + u));
+      const int there = __shfl_sync(0xffffffffu, (int)valid, 2 * (j0 + u));
       raw[u][0] = 0u;
       if constexpr (DPL == 4) raw[u][1] = 0u;
       if (dims && there) {
@@ -147,7 +150,7 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
         v[i] = __uint_as_float(i % 2 == 0 ? raw[u][i / 2] << 16 : raw[u][i / 2] & 0xffff0000u);
 #pragma unroll
       for (int h = 0; h < PER; ++h) {
-        const float pv = __shfl_sync(0xffffffffu, pj[h], j0 + u);
+        const float pv = __shfl_sync(0xffffffffu, pj[h], 2 * (j0 + u));
 #pragma unroll
         for (int i = 0; i < DPL; ++i) acc[h][i] = fmaf(pv, v[i], acc[h][i]);
       }
@@ -165,7 +168,7 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
 #pragma unroll
     for (int i = 0; i < DPL; ++i) acc_s[warp][h][lane * DPL + i] = acc[h][i];
   __syncthreads();
-  // the four warps' results as one: thread per (head, value dim)
+  // the warps' results as one: thread per (head, value dim)
   for (int e = threadIdx.x; e < per * vd; e += 32 * kWarps) {
     const int h = e / vd, d = e % vd;
     float m = -INFINITY;

@@ -97,11 +97,18 @@ static __global__ void channel_carry_kernel(float* __restrict__ scratch, const f
   if (slot < 0) return;
   const int n = cu_new[s + 1] - cu_new[s];
   float S = seq_start[s] > 0 ? state[(size_t)slot * width + c] : 0.f;
-  for (int p = 0; p < pieces && p * piece < n; ++p) {
-    float* mine = scratch + (((size_t)s * pieces + p) * width + c) * 2;
-    const float A = mine[0], B = mine[1];
-    mine[1] = S;
-    S = fmaf(A, S, B);
+  const int count = min(pieces, (n + piece - 1) / piece);
+  float2* mine = reinterpret_cast<float2*>(scratch) + (size_t)s * pieces * width + c;
+  constexpr int kAhead = 8;      // pieces asked for at a time
+  for (int p0 = 0; p0 < count; p0 += kAhead) {
+    float2 ab[kAhead];
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) ab[u] = p0 + u < count ? mine[(size_t)(p0 + u) * width] : make_float2(1.f, 0.f);
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+      if (p0 + u < count) mine[(size_t)(p0 + u) * width].y = S;
+      S = fmaf(ab[u].x, S, ab[u].y);
+    }
   }
 }
 
