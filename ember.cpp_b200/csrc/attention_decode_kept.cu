@@ -11,7 +11,8 @@
 // they use the first, so that a block waits for memory a few times and not once a key.  Softmax, sums and accumulators are
 // float32.  Partial results (m, l, acc[vd]) per (token, head, chunk) go to scratch that the caller gives.
 // With `slopes` the score of key j loses slopes[head] * (p - j); with `sinks` the merge adds exp(sinks[head]) to the
-// softmax's denominator (a term without a key or a value).
+// softmax's denominator (a term without a key or a value).  With `dist_bias` a score gains its head's entry for the
+// distance to the key.
 #include "common.cuh"
 
 namespace {
@@ -28,7 +29,7 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
                            const int* __restrict__ positions, const int* __restrict__ seq_slot,
                            const int* __restrict__ pages, int max_blocks, int n_heads, int kv_heads, int hd, int vd,
                            float scale, int window, int keep_first, int n_chunks, const float* __restrict__ slopes, int chunk,
-                           const float* __restrict__ head_scales) {
+                           const float* __restrict__ head_scales, const float* __restrict__ dist_bias, int n_dist) {
   __shared__ __align__(16) float q_s[PER][256];
   __shared__ float m_s[kWarps][PER], l_s[kWarps][PER];
   __shared__ float acc_s[kWarps][PER][32 * DPL];
@@ -105,7 +106,8 @@ decode_kept_partial_kernel(const __nv_bfloat16* __restrict__ qkv, const __nv_bfl
     const float slope = slopes && h < per ? slopes[g * per + h] : 0.f;
     const float hs = head_scales && h < per ? scale * head_scales[g * per + h] : scale;
     sc[h] += __shfl_xor_sync(0xffffffffu, sc[h], 1);
-    const float s = valid ? sc[h] * hs - slope * (float)(p - j) : -INFINITY;
+    const float near = dist_bias && valid && h < per ? dist_bias[(size_t)(g * per + h) * n_dist + min(p - j, n_dist - 1)] : 0.f;
+    const float s = valid ? sc[h] * hs - slope * (float)(p - j) + near : -INFINITY;
     const float m = warp_max(s);  // (the warp's first key is always there: m is finite)
     pj[h] = valid ? expf(s - m) : 0.f;
     const float l = 0.5f * warp_sum(pj[h]);     // (every key counts in two lanes)
@@ -240,10 +242,11 @@ template <int PER, int DPL>
 void launch_partial(dim3 grid, cudaStream_t stream, const void* qkv, const void* kc, const void* vc, float* part,
                     const int* positions, const int* seq_slot, const int* pages, int max_blocks, int n_heads,
                     int kv_heads, int hd, int vd, float scale, int window, int keep_first, int n_chunks, const float* slopes,
-                    int chunk, const float* head_scales) {
+                    int chunk, const float* head_scales, const float* dist_bias, int n_dist) {
   launch_plain(decode_kept_partial_kernel<PER, DPL>, grid, dim3(32 * kWarps), 0, stream, (const __nv_bfloat16*)qkv,
              (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, part, positions, seq_slot, pages, max_blocks, n_heads,
-             kv_heads, hd, vd, scale, window, keep_first, n_chunks, slopes, chunk, head_scales);
+             kv_heads, hd, vd, scale, window, keep_first, n_chunks, slopes, chunk, head_scales,
+             dist_bias, n_dist);
 }
 
 }  // namespace
@@ -279,7 +282,7 @@ EMBER_API int ember_attention_decode_chunked(const void* qkv, const void* kc, co
                                              const int* positions, const int* seq_slot, const int* pages, int max_blocks,
                                              int T, int n_heads, int kv_heads, int hd, int vd, float scale, int window,
                                              int keep_first, int max_keys, const float* slopes, const float* sinks, int chunk,
-                                             const float* head_scales, cudaStream_t stream);
+                                             const float* head_scales, const float* dist_bias, int n_dist, cudaStream_t stream);
 
 EMBER_API int ember_attention_decode_biased(const void* qkv, const void* kc, const void* vc, void* out, float* scratch,
                                             const int* positions, const int* seq_slot, const int* pages, int max_blocks,
@@ -287,22 +290,24 @@ EMBER_API int ember_attention_decode_biased(const void* qkv, const void* kc, con
                                             int keep_first, int max_keys, const float* slopes, const float* sinks,
                                             cudaStream_t stream) {
   return ember_attention_decode_chunked(qkv, kc, vc, out, scratch, positions, seq_slot, pages, max_blocks, T, n_heads, kv_heads,
-                                        hd, vd, scale, window, keep_first, max_keys, slopes, sinks, 0, nullptr, stream);
+                                        hd, vd, scale, window, keep_first, max_keys, slopes, sinks, 0, nullptr, nullptr, 0, stream);
 }
 
 // The same with sight limited to the query's own chunk (chunk > 0, in place of a window) and one more factor on the
-// scores of every query head (head_scales: float32 per query head, or null).
+// scores of every query head (head_scales: float32 per query head, or null).  dist_bias: float32 [heads, n_dist] or null:
+// what a score gains by the distance to the key, distances from n_dist - 1 on taking the last column.
 EMBER_API int ember_attention_decode_chunked(const void* qkv, const void* kc, const void* vc, void* out, float* scratch,
                                              const int* positions, const int* seq_slot, const int* pages, int max_blocks,
                                              int T, int n_heads, int kv_heads, int hd, int vd, float scale, int window,
                                              int keep_first, int max_keys, const float* slopes, const float* sinks, int chunk,
-                                             const float* head_scales, cudaStream_t stream) {
+                                             const float* head_scales, const float* dist_bias, int n_dist, cudaStream_t stream) {
   EMBER_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "attention_decode_kept: chunk %d beside window %d",
               chunk, window);
   EMBER_CHECK(T > 0 && n_heads > 0 && kv_heads > 0 && max_blocks > 0 && max_keys > 0, "attention_decode_kept: bad sizes");
   EMBER_CHECK(n_heads % kv_heads == 0, "attention_decode_kept: %d heads are not a multiple of %d key/value heads", n_heads,
               kv_heads);
   EMBER_CHECK(window >= 0 && keep_first >= 0, "attention_decode_kept: window %d, kept first %d", window, keep_first);
+  EMBER_CHECK(dist_bias == nullptr || n_dist > 0, "attention_decode_kept: a bias for %d distances", n_dist);
   const int per = n_heads / kv_heads;
   int dpl = 0;
   for (int cand = 1; cand <= 4; cand *= 2)
@@ -314,7 +319,7 @@ EMBER_API int ember_attention_decode_chunked(const void* qkv, const void* kc, co
   const int per_up = per <= 1 ? 1 : per <= 2 ? 2 : per <= 4 ? 4 : 8;
 #define EMBER_KEPT(PER, DPL)                                                                                              \
   launch_partial<PER, DPL>(grid, stream, qkv, kc, vc, scratch, positions, seq_slot, pages, max_blocks, n_heads, kv_heads, \
-                           hd, vd, scale, window, keep_first, n_chunks, slopes, chunk, head_scales)
+                           hd, vd, scale, window, keep_first, n_chunks, slopes, chunk, head_scales, dist_bias, n_dist)
 #define EMBER_KEPT_PER(PER)          \
   do {                               \
     if (dpl == 1) EMBER_KEPT(PER, 1); \

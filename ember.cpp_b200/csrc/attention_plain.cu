@@ -141,7 +141,7 @@ attention_plain_kernel(const T* __restrict__ qkv, const T* __restrict__ kc, cons
                        const int* __restrict__ seq_slot, const int* __restrict__ pages, int max_blocks, int T_tokens,
                        int n_heads, int kv_heads, int hd, float scale_all, int window, int vd, int keep_first,
                        const float* __restrict__ slopes, const float* __restrict__ sinks, int chunk,
-                       const float* __restrict__ head_scales) {
+                       const float* __restrict__ head_scales, const float* __restrict__ dist_bias, int n_dist) {
   __shared__ float q_s[4][kMaxHeadDim];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int item = blockIdx.x * 4 + warp;
@@ -187,6 +187,7 @@ attention_plain_kernel(const T* __restrict__ qkv, const T* __restrict__ kc, cons
       float dot = 0.f;
       for (int d = 0; d < hd; ++d) dot = fmaf(q_s[warp][d], to_float(k[d]), dot);
       sc = dot * scale - slope * (float)(p - j);
+      if (dist_bias) sc += dist_bias[(size_t)h * n_dist + min(p - j, n_dist - 1)];
     }
     const float m_new = fmaxf(m, warp_max(sc));
     const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
@@ -244,25 +245,27 @@ EMBER_API int ember_attention_plain_chunked(const void* qkv, const void* kc, con
                                             const int* token_seq, const int* seq_slot, const int* pages, int max_blocks, int T,
                                             int n_heads, int kv_heads, int hd, float scale, int window, int vd, int keep_first,
                                             const float* slopes, const float* sinks, int chunk, const float* head_scales,
-                                            int dtype, cudaStream_t stream);
+                                            const float* dist_bias, int n_dist, int dtype, cudaStream_t stream);
 
 EMBER_API int ember_attention_plain_biased(const void* qkv, const void* kc, const void* vc, void* out, const int* positions,
                                            const int* token_seq, const int* seq_slot, const int* pages, int max_blocks, int T,
                                            int n_heads, int kv_heads, int hd, float scale, int window, int vd, int keep_first,
                                            const float* slopes, const float* sinks, int dtype, cudaStream_t stream) {
   return ember_attention_plain_chunked(qkv, kc, vc, out, positions, token_seq, seq_slot, pages, max_blocks, T, n_heads, kv_heads,
-                                       hd, scale, window, vd, keep_first, slopes, sinks, 0, nullptr, dtype, stream);
+                                       hd, scale, window, vd, keep_first, slopes, sinks, 0, nullptr, nullptr, 0, dtype, stream);
 }
 
 // The same with sight limited to the query's own chunk (chunk > 0, in place of a window: query p sees key j <= p
 // with floor(j / chunk) = floor(p / chunk)) and one more factor on the scores of every query head (head_scales:
-// float32 per query head, or null).
+// float32 per query head, or null).  dist_bias: float32 [heads, n_dist] or null: what a score gains by the distance p - j to
+// the key, distances from n_dist - 1 on taking the last column.
 EMBER_API int ember_attention_plain_chunked(const void* qkv, const void* kc, const void* vc, void* out, const int* positions,
                                             const int* token_seq, const int* seq_slot, const int* pages, int max_blocks, int T,
                                             int n_heads, int kv_heads, int hd, float scale, int window, int vd, int keep_first,
                                             const float* slopes, const float* sinks, int chunk, const float* head_scales,
-                                            int dtype, cudaStream_t stream) {
+                                            const float* dist_bias, int n_dist, int dtype, cudaStream_t stream) {
   EMBER_CHECK(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "attention: chunk %d beside window %d", chunk, window);
+  EMBER_CHECK(dist_bias == nullptr || n_dist > 0, "attention: a bias for %d distances", n_dist);
   EMBER_CHECK(T > 0 && n_heads > 0 && kv_heads > 0 && max_blocks > 0, "attention: bad sizes");
   EMBER_CHECK(n_heads % kv_heads == 0, "attention: %d heads are not a multiple of %d key/value heads", n_heads,
               kv_heads);
@@ -274,12 +277,13 @@ EMBER_API int ember_attention_plain_chunked(const void* qkv, const void* kc, con
   if (dtype == EMBER_F32)
     attention_plain_kernel<float><<<grid, 128, 0, stream>>>((const float*)qkv, (const float*)kc, (const float*)vc,
                                                             (float*)out, positions, token_seq, seq_slot, pages,
-                                                            max_blocks, T, n_heads, kv_heads, hd, scale, window, vd, keep_first, slopes, sinks, chunk, head_scales);
+                                                            max_blocks, T, n_heads, kv_heads, hd, scale, window, vd, keep_first, slopes, sinks, chunk, head_scales,
+                                                            dist_bias, n_dist);
   else if (dtype == EMBER_BF16)
     attention_plain_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(
         (const __nv_bfloat16*)qkv, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, (__nv_bfloat16*)out, positions,
         token_seq, seq_slot, pages, max_blocks, T, n_heads, kv_heads, hd, scale, window, vd, keep_first, slopes, sinks, chunk,
-        head_scales);
+        head_scales, dist_bias, n_dist);
   else
     return ember_fail("attention: element type %d", dtype);
   EMBER_LAUNCH_OK("attention_plain");

@@ -132,7 +132,7 @@ __global__ void layernorm_kernel(const float* __restrict__ x, const float* __res
       const int i = lane + 32 * j;
       if (i < (d >> 2)) {
         gm_early[j] = reinterpret_cast<const float4*>(w)[i];
-        bt_early[j] = reinterpret_cast<const float4*>(b)[i];
+        bt_early[j] = b ? reinterpret_cast<const float4*>(b)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
       }
     }
   }
@@ -168,7 +168,7 @@ __global__ void layernorm_kernel(const float* __restrict__ x, const float* __res
       const int i = lane + 32 * j;
       if (i < nv) {
         const float4 gm = EARLY ? gm_early[j] : reinterpret_cast<const float4*>(w)[i];
-        const float4 bt = EARLY ? bt_early[j] : reinterpret_cast<const float4*>(b)[i];
+        const float4 bt = EARLY ? bt_early[j] : b ? reinterpret_cast<const float4*>(b)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
         store4<OutT>(o + 4 * i, (v[j].x - mean) * inv * gm.x + bt.x, (v[j].y - mean) * inv * gm.y + bt.y,
                      (v[j].z - mean) * inv * gm.z + bt.z, (v[j].w - mean) * inv * gm.w + bt.w);
       }
@@ -186,7 +186,7 @@ __global__ void layernorm_kernel(const float* __restrict__ x, const float* __res
   }
   const float var = warp_sum(q) / (float)d;
   const float inv = 1.0f / sqrtf(var + eps);
-  for (int i = lane; i < d; i += 32) o[i] = from_float<OutT>((__ldcg(r + i) - mean) * inv * w[i] + b[i]);
+  for (int i = lane; i < d; i += 32) o[i] = from_float<OutT>((__ldcg(r + i) - mean) * inv * w[i] + (b ? b[i] : 0.f));
 }
 
 EMBER_API int ember_layernorm(const float* x, const float* w, const float* b, void* out, int rows, int d, float eps,

@@ -10,7 +10,7 @@
 //   latent_rows     per token: the query row's RMS norm, the cached row's RMS norm, the shared key
 //                   part's rotation, and the write of both into the cache, one launch
 //   head_linear     out[t, h] = a[t, h] W[h]^T for every head h, heads side by side in a row
-//   latent_attention_plain   one warp per (token, head), keys in groups of 32 from position 0, an online
+//   latent_attention_plain   one warp per (token, head), keys in groups of 32 from the first visible one, an online
 //                   softmax whose order depends on key positions alone: the kernel of the 32-bit path
 //                   and the twin that the faster kernels are tested against
 #include "common.cuh"
@@ -58,12 +58,12 @@ __global__ void rotate_kernel(const TS* src, long long src_stride, int src_col, 
   for (int i = dims + threadIdx.x; i < width; i += blockDim.x) d[i] = from_float<TD>(to_float(s[i]));
 }
 
-// grid (T): down float32 [T, q_rank (+ rank + rot)].
+// grid (T): down float32 [T, down_width], of which q_rank (+ rank + rot) columns are read.
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
 latent_rows_kernel(const float* __restrict__ down, int down_width, int q_rank, const float* __restrict__ q_gain,
                    const float* __restrict__ c_gain, int rank, int rot, float eps, const float* __restrict__ freqs,
-                   float magnitude, int dims, T* __restrict__ c_q, T* __restrict__ kc, T* __restrict__ vc,
+                   float magnitude, int dims, int interleaved, T* __restrict__ c_q, T* __restrict__ kc, T* __restrict__ vc,
                    const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ seq_slot,
                    const int* __restrict__ pages, int max_blocks) {
   __shared__ float red[kThreads / 32];
@@ -94,9 +94,10 @@ latent_rows_kernel(const float* __restrict__ down, int down_width, int q_rank, c
   const int half = dims / 2;
   for (int i = threadIdx.x; i < half; i += kThreads) {
     float ou, ov;
-    turn(r[i], r[i + half], p, freqs[i], magnitude, ou, ov);
-    vdst[i] = from_float<T>(ou);
-    vdst[i + half] = from_float<T>(ov);
+    const int iu = interleaved ? 2 * i : i, iv = interleaved ? 2 * i + 1 : i + half;
+    turn(r[iu], r[iv], p, freqs[i], magnitude, ou, ov);
+    vdst[iu] = from_float<T>(ou);
+    vdst[iv] = from_float<T>(ov);
   }
   for (int i = dims + threadIdx.x; i < rot; i += kThreads) vdst[i] = from_float<T>(r[i]);
 }
@@ -144,7 +145,7 @@ __global__ void __launch_bounds__(128)
 latent_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc, T* __restrict__ out,
                               const int* __restrict__ positions, const int* __restrict__ token_seq,
                               const int* __restrict__ seq_slot, const int* __restrict__ pages, int max_blocks, int T_tokens,
-                              int heads, int rank, int rot, float scale) {
+                              int heads, int rank, int rot, float scale, int window) {
   extern __shared__ float q_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int item = blockIdx.x * 4 + warp;
@@ -168,10 +169,11 @@ latent_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ kc,
   float acc[kMaxRank / 32];
 #pragma unroll
   for (int i = 0; i < kMaxRank / 32; ++i) acc[i] = 0.f;
-  const int n_keys = p + 1;
+  const int lo = window > 0 ? max(0, p - window + 1) : 0;   // the first visible position
+  const int n_keys = p + 1 - lo;
   for (int base = 0; base < n_keys; base += 32) {
-    const int j = base + lane;
-    const int page = j < n_keys ? my_pages[j / kPage] : -1;
+    const int j = lo + base + lane;
+    const int page = base + lane < n_keys ? my_pages[j / kPage] : -1;
     const bool valid = page >= 0;   // a page that is not held contributes nothing and is never read
     size_t r = 0;
     float sc = -INFINITY;
@@ -253,23 +255,23 @@ EMBER_API int ember_rotate_pairs(const void* src, long long src_stride, int src_
 
 // kc, vc null: a layer that reads another's cached rows makes only its query row.
 EMBER_API int ember_latent_rows(const float* down, int down_width, int q_rank, const float* q_gain, const float* c_gain,
-                                int rank, int rot, float eps, const float* freqs, float magnitude, int dims, void* c_q,
-                                void* kc, void* vc, const int* positions, const int* token_seq, const int* seq_slot,
+                                int rank, int rot, float eps, const float* freqs, float magnitude, int dims, int interleaved,
+                                void* c_q, void* kc, void* vc, const int* positions, const int* token_seq, const int* seq_slot,
                                 const int* pages, int max_blocks, int T, int dtype, cudaStream_t stream) {
   EMBER_CHECK(T > 0 && q_rank > 0 && down_width >= q_rank, "latent_rows: bad sizes");
   EMBER_CHECK((kc == nullptr) == (vc == nullptr), "latent_rows: both cache tensors or none");
   if (kc != nullptr) {
-    EMBER_CHECK(rank > 0 && rot > 0 && down_width == q_rank + rank + rot, "latent_rows: rows of %d are not %d + %d + %d",
+    EMBER_CHECK(rank > 0 && rot > 0 && down_width >= q_rank + rank + rot, "latent_rows: rows of %d are less than %d + %d + %d",
                 down_width, q_rank, rank, rot);
     EMBER_CHECK(dims > 0 && dims % 2 == 0 && dims <= rot, "latent_rows: %d rotated dimensions of %d", dims, rot);
   }
   if (dtype == EMBER_F32)
     latent_rows_kernel<float><<<T, kThreads, 0, stream>>>(down, down_width, q_rank, q_gain, c_gain, rank, rot, eps, freqs,
-                                                          magnitude, dims, (float*)c_q, (float*)kc, (float*)vc, positions,
+                                                          magnitude, dims, interleaved, (float*)c_q, (float*)kc, (float*)vc, positions,
                                                           token_seq, seq_slot, pages, max_blocks);
   else if (dtype == EMBER_BF16)
     latent_rows_kernel<__nv_bfloat16><<<T, kThreads, 0, stream>>>(
-        down, down_width, q_rank, q_gain, c_gain, rank, rot, eps, freqs, magnitude, dims, (__nv_bfloat16*)c_q,
+        down, down_width, q_rank, q_gain, c_gain, rank, rot, eps, freqs, magnitude, dims, interleaved, (__nv_bfloat16*)c_q,
         (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, positions, token_seq, seq_slot, pages, max_blocks);
   else
     return ember_fail("latent_rows: element type %d", dtype);
@@ -297,8 +299,9 @@ EMBER_API int ember_head_linear(const void* a, long long a_stride, int a_col, in
 
 EMBER_API int ember_latent_attention_plain(const void* q, const void* kc, const void* vc, void* out, const int* positions,
                                            const int* token_seq, const int* seq_slot, const int* pages, int max_blocks, int T,
-                                           int heads, int rank, int rot, float scale, int dtype, cudaStream_t stream) {
+                                           int heads, int rank, int rot, float scale, int window, int dtype, cudaStream_t stream) {
   EMBER_CHECK(T > 0 && heads > 0 && max_blocks > 0, "latent_attention: bad sizes");
+  EMBER_CHECK(window >= 0, "latent_attention: window %d", window);
   EMBER_CHECK(rank >= 1 && rank <= kMaxRank && rot >= 1, "latent_attention: rows of %d + %d values (at most %d + any)", rank,
               rot, kMaxRank);
   const long long items = (long long)T * heads;
@@ -308,11 +311,11 @@ EMBER_API int ember_latent_attention_plain(const void* q, const void* kc, const 
   if (dtype == EMBER_F32)
     latent_attention_plain_kernel<float><<<grid, 128, smem, stream>>>((const float*)q, (const float*)kc, (const float*)vc,
                                                                       (float*)out, positions, token_seq, seq_slot, pages,
-                                                                      max_blocks, T, heads, rank, rot, scale);
+                                                                      max_blocks, T, heads, rank, rot, scale, window);
   else if (dtype == EMBER_BF16)
     latent_attention_plain_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, (__nv_bfloat16*)out, positions, token_seq,
-        seq_slot, pages, max_blocks, T, heads, rank, rot, scale);
+        seq_slot, pages, max_blocks, T, heads, rank, rot, scale, window);
   else
     return ember_fail("latent_attention: element type %d", dtype);
   EMBER_LAUNCH_OK("latent_attention_plain");

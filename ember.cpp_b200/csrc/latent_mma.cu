@@ -8,7 +8,7 @@
 // keys; they tell each other their rows' maxima and hand each other their probabilities (bfloat16)
 // through shared memory, meeting at a barrier of their own, and each adds P C for all 64 keys to its own
 // half of the output's `rank` columns, which stays in registers (up to 128 float32 values a thread).
-// Keys past a row's own position are masked by selection; float32 softmax in base 2.
+// Keys past a row's own position, or before its window, are masked by selection; float32 softmax in base 2.
 //
 // One token a sequence (a decode step): the pages are cut into chunks, a block a chunk (grid z); blocks
 // leave unnormalised sums with their maximum and total, and `latent_merge` combines them.  Otherwise
@@ -58,7 +58,7 @@ __global__ void __launch_bounds__(256, 1)
 latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc, bf16* __restrict__ out,
                   float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ seq_slot,
                   const int* __restrict__ seq_start, const int* __restrict__ cu_new, const int* __restrict__ pages,
-                  int max_blocks, int heads, int rank, int rot, float scale_log2, int ppc, int n_chunks) {
+                  int max_blocks, int heads, int rank, int rot, float scale_log2, int window, int ppc, int n_chunks) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int W = rank + rot, WS = W + 8, vecs = W / 8;
   const int G = blockDim.x >> 6;
@@ -78,7 +78,9 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const
   const int slot = seq_slot[s];
   const int start = seq_start[s];
   const int p_max = start + (min(R, r0 + 16 * G) - 1) / heads;
-  const int pg0 = chunk * ppc, pg1 = min(pg0 + ppc, p_max / kPage + 1);
+  // the block's pages: from the one that holds the first position its first row sees
+  const int pg0 = (window > 0 ? max(0, start + r0 / heads - window + 1) / kPage : 0) + chunk * ppc;
+  const int pg1 = min(pg0 + ppc, p_max / kPage + 1);
   if (slot < 0 || pg0 >= pg1) {   // padding, or a chunk past this block's rows: nothing to add
     if (n_chunks == 1) {
       for (int i = threadIdx.x; i < 16 * G * rank; i += blockDim.x) {
@@ -100,6 +102,7 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const
       *reinterpret_cast<uint4*>(qs + (size_t)row * WS + v * 8) = make_uint4(0, 0, 0, 0);
   }
   const int pa_row = start + ra / heads, pb_row = start + rb / heads;   // the rows' own positions
+  const int span = window > 0 ? window : 0x40000000;      // how many positions a row sees
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
   float o_acc[RMAX / 16][4];
 #pragma unroll
@@ -141,7 +144,7 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const
       for (int e = 0; e < 4; ++e) {
         const int j = pg * kPage + half * 32 + nt * 8 + 2 * (lane & 3) + (e & 1);
         const bool top = e < 2;
-        const bool seen = page >= 0 && (top ? (ra < R && j <= pa_row) : (rb < R && j <= pb_row));
+        const bool seen = page >= 0 && (top ? (ra < R && j <= pa_row && j > pa_row - span) : (rb < R && j <= pb_row && j > pb_row - span));
         const float v = seen ? sa[nt][e] * scale_log2 : -INFINITY;
         sa[nt][e] = v;
         if (top) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
@@ -282,12 +285,12 @@ EMBER_API size_t ember_latent_attention_mma_scratch(int rows, int rank, int n_ch
 }
 
 // Returns 2 (and launches nothing) for sizes that this kernel has no form for.  q bfloat16 [T, heads * (rank + rot)],
-// out bfloat16 [T, heads * rank]; n_chunks > 1 only with one token a sequence; scratch as the function above says.
+// out bfloat16 [T, heads * rank]; window 0: all keys; the chunks count from the first page that a row sees; n_chunks > 1 only with one token a sequence; scratch as the function above says.
 EMBER_API int ember_latent_attention_mma(const void* q, const void* kc, const void* vc, void* out, float* scratch,
                                          const int* seq_slot, const int* seq_start, const int* cu_new, const int* pages,
                                          int max_blocks, int n_seq, int max_new, int T, int heads, int rank, int rot, float scale,
-                                         int n_chunks, int pages_per_chunk, cudaStream_t stream) {
-  EMBER_CHECK(n_seq > 0 && max_new > 0 && heads > 0 && max_blocks > 0 && n_chunks >= 1 && pages_per_chunk >= 1,
+                                         int window, int n_chunks, int pages_per_chunk, cudaStream_t stream) {
+  EMBER_CHECK(n_seq > 0 && max_new > 0 && heads > 0 && max_blocks > 0 && n_chunks >= 1 && pages_per_chunk >= 1 && window >= 0,
               "latent_attention_mma: bad sizes");
   if (rank % 32 != 0 || rank > 512 || rot % 16 != 0 || rot <= 0 || !(scale > 0.f)) return 2;
   EMBER_CHECK(n_chunks == 1 || max_new == 1, "latent_attention_mma: chunks are for steps of one token a sequence");
@@ -313,7 +316,7 @@ EMBER_API int ember_latent_attention_mma(const void* q, const void* kc, const vo
     }                                                                                                                     \
     latent_mma_kernel<RMAX><<<grid, 64 * G, smem, stream>>>((const bf16*)q, (const bf16*)kc, (const bf16*)vc, (bf16*)out, part_o, \
                                                             part_ml, seq_slot, seq_start, cu_new, pages, max_blocks, heads, rank, \
-                                                            rot, scale_log2, pages_per_chunk, n_chunks);                  \
+                                                            rot, scale_log2, window, pages_per_chunk, n_chunks);          \
   } while (0)
   if (smem > 200 * 1024) return 2;
   if (rank <= 128)

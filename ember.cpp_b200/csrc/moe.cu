@@ -6,6 +6,7 @@
 // pairs in expert order (sorted[pairs]; the order inside an expert is whatever the atomics gave, which no
 // result depends on: every pair's row is computed by itself).  The products:
 //   gate_up   inner[q, :] = silu(Wg_e a_t) * (Wu_e a_t)     (W_e = [gate | up] stacked, [2 * inner, width])
+//   up        inner[q, :] = act(Wu_e a_t)                   (experts without a gate: W_e [inner, width])
 //   down      y[q, :]     = Wd_e inner[q, :]                (float32)
 // Few pairs (a decode step): a warp per output value streams the expert's rows once, which is all the
 // traffic there is.  Many pairs (a prompt): tiles of one expert's pairs and outputs on mma.sync
@@ -98,6 +99,22 @@ moe_gate_up_stream_kernel(const T* __restrict__ a, const T* __restrict__ w, cons
   }
 }
 
+// grid (pairs, ceil(inner / 32)): an expert without a gate, act an activation code
+template <typename T>
+__global__ void __launch_bounds__(kStreamWarps * 32)
+moe_up_stream_kernel(const T* __restrict__ a, const T* __restrict__ w, const int* __restrict__ pair_expert, T* __restrict__ out,
+                     int top, int width, int inner, int act) {
+  const int q = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* row = a + (size_t)(q / top) * width;
+  const T* we = w + (size_t)pair_expert[q] * inner * width;
+  for (int i = 0; i < kStreamOutputs; ++i) {
+    const int f = (blockIdx.y * kStreamWarps + warp) * kStreamOutputs + i;
+    if (f >= inner) return;
+    const float v = warp_dot(we + (size_t)f * width, row, width, lane);
+    if (lane == 0) out[(size_t)q * inner + f] = from_float<T>(apply_act(v, act));
+  }
+}
+
 // grid (pairs, ceil(width / 32))
 template <typename T>
 __global__ void __launch_bounds__(kStreamWarps * 32)
@@ -139,20 +156,24 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const unsigned (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <bool GATED>
+enum : int { kFormDown = 0, kFormGated = 1, kFormUp = 2 };
+
+template <int FORM>
 constexpr int tile_smem() {
-  return (2 * kTileM * kLd + 2 * (GATED ? 2 : 1) * kTileN * kLd) * (int)sizeof(__nv_bfloat16);
+  return (2 * kTileM * kLd + 2 * (FORM == kFormGated ? 2 : 1) * kTileN * kLd) * (int)sizeof(__nv_bfloat16);
 }
 
-// GATED: W_e = [gate | up] of n_out rows each, the result silu(gate) * up in bfloat16 and the input rows are
-// the tokens' (pair / top); else W_e has n_out rows, the result is float32 and the input rows are the pairs'.
+// kFormGated: W_e = [gate | up] of n_out rows each, the result silu(gate) * up in bfloat16 and the input rows are the
+// tokens' (pair / top); kFormUp: W_e has n_out rows, the result act(W_e a) in bfloat16, the input rows the tokens'; kFormDown:
+// W_e has n_out rows, the result is float32 and the input rows are the pairs'.
 // grid (tiles of pairs: an upper bound, ceil(n_out / 64)); a block finds its expert and its tile of that
 // expert's pairs from the offsets, and leaves if there is none.  Four warps, each 32 pairs x 64 outputs.
-template <bool GATED>
+template <int FORM>
 __global__ void __launch_bounds__(128)
 moe_tile_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w, const int* __restrict__ offsets,
                 const int* __restrict__ sorted, void* __restrict__ out, int experts, int top, int K, int n_out, float limit,
-                float alpha, float shift) {
+                float alpha, float shift, int act) {
+  constexpr bool GATED = FORM == kFormGated;
   constexpr int NW = GATED ? 2 : 1;
   extern __shared__ __align__(16) unsigned char tile_raw[];
   __nv_bfloat16* sA = reinterpret_cast<__nv_bfloat16*>(tile_raw);  // [2][kTileM * kLd]
@@ -181,7 +202,7 @@ moe_tile_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __rest
   {
     const int q = (int)threadIdx.x < count ? sorted[first + threadIdx.x] : -1;
     s_pair[threadIdx.x] = q;
-    s_rows[threadIdx.x] = q < 0 ? -1 : (GATED ? q / top : q);
+    s_rows[threadIdx.x] = q < 0 ? -1 : (FORM != kFormDown ? q / top : q);
   }
   __syncthreads();
 
@@ -274,6 +295,13 @@ moe_tile_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __rest
             *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(y0, y1);
           else
             *dst = __float2bfloat16_rn(y0);
+        } else if constexpr (FORM == kFormUp) {
+          const float y0 = apply_act(acc[0][f][i][2 * r], act), y1 = apply_act(acc[0][f][i][2 * r + 1], act);
+          __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(out) + (size_t)q * n_out + n;
+          if (n + 1 < n_out)
+            *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(y0, y1);
+          else
+            *dst = __float2bfloat16_rn(y0);
         } else {
           float* dst = static_cast<float*>(out) + (size_t)q * n_out + n;
           if (n + 1 < n_out)
@@ -286,28 +314,28 @@ moe_tile_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __rest
   }
 }
 
-template <bool GATED>
+template <int FORM>
 int launch_tiles(const void* a, const void* w, const int* offsets, const int* sorted, void* out, long long pairs, int experts,
                  int top, int K, int n_out, cudaStream_t stream, const char* name, float limit = 0.f, float alpha = 1.f,
-                 float shift = 0.f) {
+                 float shift = 0.f, int act = EMBER_ACT_NONE) {
   static bool configured = false;  // per instantiation
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(moe_tile_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, tile_smem<GATED>());
+    cudaError_t e = cudaFuncSetAttribute(moe_tile_kernel<FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, tile_smem<FORM>());
     if (e != cudaSuccess) return ember_fail("%s: %s", name, cudaGetErrorString(e));
     configured = true;
   }
   const dim3 grid((unsigned)((pairs + kTileM - 1) / kTileM + experts), (n_out + kTileN - 1) / kTileN);
   EMBER_CHECK(grid.y <= 65535, "%s: %d outputs exceed one launch", name, n_out);
-  moe_tile_kernel<GATED><<<grid, 128, tile_smem<GATED>(), stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w, offsets,
-                                                                    sorted, out, experts, top, K, n_out, limit, alpha, shift);
+  moe_tile_kernel<FORM><<<grid, 128, tile_smem<FORM>(), stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w, offsets, sorted,
+                                                                  out, experts, top, K, n_out, limit, alpha, shift, act);
   EMBER_LAUNCH_OK(name);
   return 0;
 }
 
 // ---------------------------------------------------------------------------- the router's choice
 // A warp a token.  s = sigmoid(z); the choice is made on s + correction among the experts of the `keep` groups
-// whose two largest choice scores add up to the most; weights = s of the chosen, over their sum (+ 1e-20), times
-// `scale`.  Among equal scores the lower index wins.  Dynamic shared memory: per warp 2 * experts + groups floats.
+// whose `group_top` (2 or 1) largest choice scores add up to the most; weights = s of the chosen, over their sum (+ 1e-20),
+// times `scale`.  kScoresAll: s = softmax(z) over all experts, weights = s of the chosen times `scale`.  Among equal scores the lower index wins.  Dynamic shared memory: per warp 2 * experts + groups floats.
 constexpr int kPickWarps = 4;
 
 __device__ __forceinline__ void warp_argmax(float& best, int& at) {
@@ -322,9 +350,11 @@ __device__ __forceinline__ void warp_argmax(float& best, int& at) {
   }
 }
 
+enum : int { kScoresSigmoid = 0, kScoresChosen = 1, kScoresAll = 2 };
+
 __global__ void __launch_bounds__(32 * kPickWarps)
 moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int T, int experts, int top,
-                int groups, int keep, float scale, int softmax, int* __restrict__ chosen, float* __restrict__ weights) {
+                int groups, int keep, int group_top, float scale, int scores, int* __restrict__ chosen, float* __restrict__ weights) {
   extern __shared__ float pick_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kPickWarps + warp;
@@ -332,10 +362,18 @@ moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restric
   float* sc = pick_sm + (size_t)warp * (2 * experts + groups);
   float* ch = sc + experts;
   float* gs = ch + experts;
+  const bool softmax = scores == kScoresChosen;
+  float top_z = -INFINITY, all = 0.f;
+  if (scores == kScoresAll) {
+    for (int e = lane; e < experts; e += 32) top_z = fmaxf(top_z, logits[(size_t)t * ld + e]);
+    top_z = warp_max(top_z);
+    for (int e = lane; e < experts; e += 32) all += expf(logits[(size_t)t * ld + e] - top_z);
+    all = warp_sum(all);
+  }
   for (int e = lane; e < experts; e += 32) {
-    // (softmax: the stored vector is a bias of the logits, which are chosen by and weigh as they are)
+    // (softmax over the chosen: the stored vector is a bias of the logits, which are chosen by and weigh as they are)
     const float z = logits[(size_t)t * ld + e];
-    const float s = softmax ? z + correction[e] : 1.0f / (1.0f + expf(-z));
+    const float s = softmax ? z + correction[e] : scores == kScoresAll ? expf(z - top_z) / all : 1.0f / (1.0f + expf(-z));
     sc[e] = s;
     ch[e] = softmax ? s : s + correction[e];
   }
@@ -353,7 +391,7 @@ moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restric
           m2 = v;
         }
       }
-      gs[g] = per >= 2 ? m1 + m2 : m1;
+      gs[g] = per >= 2 && group_top == 2 ? m1 + m2 : m1;
     }
     __syncwarp();
     for (int it = 0; it < keep; ++it) {     // a kept group's score becomes +inf, which is never picked again
@@ -397,15 +435,16 @@ moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restric
     }
     __syncwarp();
   }
-  const float f = scale / (sum + 1e-20f);
+  const float f = scores == kScoresAll ? scale : scale / (sum + 1e-20f);
   for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= f;
 }
 
+// rows (or null): out once more, in bfloat16.
 // grid (T): out = x + sum_k weights[t, k] y[t, k, :] (k ascending) + sigmoid(gate) * shared[t, :]
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ weights,
                    const float* __restrict__ shared, const float* __restrict__ logits, int ld, int gate_col,
-                   float* __restrict__ out, int top, int width) {
+                   float* __restrict__ out, __nv_bfloat16* __restrict__ rows, int top, int width) {
   const int t = blockIdx.x;
   const float* w = weights + (size_t)t * top;
   const float sg = shared == nullptr ? 0.f : (logits == nullptr ? 1.f : 1.0f / (1.0f + expf(-logits[(size_t)t * ld + gate_col])));
@@ -413,25 +452,29 @@ moe_combine_kernel(const float* __restrict__ x, const float* __restrict__ y, con
     float acc = 0.f;
     for (int k = 0; k < top; ++k) acc = fmaf(w[k], y[((size_t)t * top + k) * width + c], acc);
     if (shared != nullptr) acc = fmaf(sg, shared[(size_t)t * width + c], acc);
-    out[(size_t)t * width + c] = x[(size_t)t * width + c] + acc;
+    acc = x[(size_t)t * width + c] + acc;
+    out[(size_t)t * width + c] = acc;
+    if (rows != nullptr) rows[(size_t)t * width + c] = __float2bfloat16_rn(acc);
   }
 }
 
 }  // namespace
 
 // logits float32 [T, ld] (the first `experts` columns are the router's), correction float32 [experts];
-// chosen int32 [T, top], weights float32 [T, top].  softmax 0: scores sigmoid(z), chosen by score + correction, weights the
-// chosen's scores over their sum; softmax 1: chosen by z + correction, weights the softmax over the chosen's (one group).
+// chosen int32 [T, top], weights float32 [T, top].  scores 0: scores sigmoid(z), chosen by score + correction, weights the
+// chosen's scores over their sum; scores 1: chosen by z + correction, weights the softmax over the chosen's (one group);
+// scores 2: scores softmax(z) over all experts, chosen by score + correction, weights the chosen's scores.
 EMBER_API int ember_moe_pick(const float* logits, int ld, const float* correction, int T, int experts, int top, int groups,
-                             int keep, float scale, int softmax, int* chosen, float* weights, cudaStream_t stream) {
-  EMBER_CHECK(!softmax || groups == 1, "moe_pick: a softmax over the chosen with %d groups", groups);
+                             int keep, int group_top, float scale, int scores, int* chosen, float* weights, cudaStream_t stream) {
+  EMBER_CHECK(scores >= 0 && scores <= 2 && (group_top == 1 || group_top == 2), "moe_pick: scores %d, group_top %d", scores, group_top);
+  EMBER_CHECK(scores != kScoresChosen || groups == 1, "moe_pick: a softmax over the chosen with %d groups", groups);
   EMBER_CHECK(T > 0 && experts > 0 && experts <= 1024 && top >= 1 && top <= experts && ld >= experts,
               "moe_pick: %d tokens, top %d of %d experts (at most 1024)", T, top, experts);
   EMBER_CHECK(groups >= 1 && experts % groups == 0 && keep >= 1 && keep <= groups && (long long)keep * (experts / groups) >= top,
               "moe_pick: %d groups of which %d are kept do not hold %d choices", groups, keep, top);
   const size_t smem = (size_t)kPickWarps * (2 * experts + groups) * sizeof(float);
   const cudaError_t e = launch_plain(moe_pick_kernel, dim3((T + kPickWarps - 1) / kPickWarps), dim3(32 * kPickWarps), smem, stream,
-                                     logits, ld, correction, T, experts, top, groups, keep, scale, softmax, chosen, weights);
+                                     logits, ld, correction, T, experts, top, groups, keep, group_top, scale, scores, chosen, weights);
   if (e != cudaSuccess) return ember_fail("moe_pick: %s", cudaGetErrorString(e));
   return 0;
 }
@@ -439,11 +482,11 @@ EMBER_API int ember_moe_pick(const float* logits, int ld, const float* correctio
 // x, out float32 [T, width]; y float32 [T, top, width]; weights float32 [T, top]; shared float32 [T, width] or null;
 // logits float32 [T, ld] or null (then the shared rows are added as they are): the shared rows' gate is column gate_col.
 EMBER_API int ember_moe_combine(const float* x, const float* y, const float* weights, const float* shared, const float* logits,
-                                int ld, int gate_col, float* out, int T, int top, int width, cudaStream_t stream) {
+                                int ld, int gate_col, float* out, void* rows, int T, int top, int width, cudaStream_t stream) {
   EMBER_CHECK(T > 0 && top > 0 && width > 0, "moe_combine: bad sizes");
   EMBER_CHECK(logits == nullptr || (gate_col >= 0 && gate_col < ld), "moe_combine: gate column %d of %d", gate_col, ld);
   const cudaError_t e = launch_plain(moe_combine_kernel, dim3(T), dim3(256), 0, stream, x, y, weights, shared, logits, ld, gate_col,
-                                     out, top, width);
+                                     out, (__nv_bfloat16*)rows, top, width);
   if (e != cudaSuccess) return ember_fail("moe_combine: %s", cudaGetErrorString(e));
   return 0;
 }
@@ -483,7 +526,7 @@ EMBER_API int ember_moe_gate_up_act(const void* a, const void* w, const int* pai
   if (tiled) {
     EMBER_CHECK(dtype == EMBER_BF16 && width % 8 == 0 && inner % 2 == 0,
                 "moe_gate_up: tiles take bfloat16 rows that are multiples of 8 and an even number of outputs");
-    return launch_tiles<true>(a, w, offsets, sorted, out, pairs, experts, top, width, inner, stream, "moe_gate_up", limit, alpha, shift);
+    return launch_tiles<kFormGated>(a, w, offsets, sorted, out, pairs, experts, top, width, inner, stream, "moe_gate_up", limit, alpha, shift);
   }
   const dim3 grid((unsigned)pairs, (inner + kStreamWarps * kStreamOutputs - 1) / (kStreamWarps * kStreamOutputs));
   EMBER_CHECK(grid.y <= 65535, "moe_gate_up: %d outputs exceed one launch", inner);
@@ -500,6 +543,32 @@ EMBER_API int ember_moe_gate_up_act(const void* a, const void* w, const int* pai
   return 0;
 }
 
+// Experts without a gate: a [T, width] (dtype), w [experts, inner, width], out [T * top, inner] (dtype) = act(w a).
+EMBER_API int ember_moe_up(const void* a, const void* w, const int* pair_expert, const int* offsets, const int* sorted, void* out,
+                           int T, int top, int experts, int width, int inner, int act, int tiled, int dtype, cudaStream_t stream) {
+  EMBER_CHECK(T > 0 && top > 0 && experts > 0 && width > 0 && inner > 0, "moe_up: bad sizes");
+  EMBER_CHECK(act >= EMBER_ACT_NONE && act <= EMBER_ACT_RELU2, "moe_up: activation %d", act);
+  const long long pairs = (long long)T * top;
+  if (tiled) {
+    EMBER_CHECK(dtype == EMBER_BF16 && width % 8 == 0 && inner % 2 == 0,
+                "moe_up: tiles take bfloat16 rows that are multiples of 8 and an even number of outputs");
+    return launch_tiles<kFormUp>(a, w, offsets, sorted, out, pairs, experts, top, width, inner, stream, "moe_up", 0.f, 1.f, 0.f, act);
+  }
+  const dim3 grid((unsigned)pairs, (inner + kStreamWarps * kStreamOutputs - 1) / (kStreamWarps * kStreamOutputs));
+  EMBER_CHECK(grid.y <= 65535, "moe_up: %d outputs exceed one launch", inner);
+  cudaError_t e;
+  if (dtype == EMBER_F32)
+    e = launch_plain(moe_up_stream_kernel<float>, grid, dim3(kStreamWarps * 32), 0, stream, (const float*)a, (const float*)w, pair_expert,
+                     (float*)out, top, width, inner, act);
+  else if (dtype == EMBER_BF16)
+    e = launch_plain(moe_up_stream_kernel<__nv_bfloat16>, grid, dim3(kStreamWarps * 32), 0, stream, (const __nv_bfloat16*)a,
+                     (const __nv_bfloat16*)w, pair_expert, (__nv_bfloat16*)out, top, width, inner, act);
+  else
+    return ember_fail("moe_up: element type %d", dtype);
+  if (e != cudaSuccess) return ember_fail("moe_up: %s", cudaGetErrorString(e));
+  return 0;
+}
+
 // a [T * top, inner] (dtype), w [experts, width, inner], out float32 [T * top, width]
 EMBER_API int ember_moe_down(const void* a, const void* w, const int* pair_expert, const int* offsets, const int* sorted,
                              float* out, int T, int top, int experts, int width, int inner, int tiled, int dtype,
@@ -509,7 +578,7 @@ EMBER_API int ember_moe_down(const void* a, const void* w, const int* pair_exper
   if (tiled) {
     EMBER_CHECK(dtype == EMBER_BF16 && inner % 8 == 0 && width % 2 == 0,
                 "moe_down: tiles take bfloat16 rows that are multiples of 8 and an even number of outputs");
-    return launch_tiles<false>(a, w, offsets, sorted, out, pairs, experts, top, inner, width, stream, "moe_down");
+    return launch_tiles<kFormDown>(a, w, offsets, sorted, out, pairs, experts, top, inner, width, stream, "moe_down");
   }
   const dim3 grid((unsigned)pairs, (width + kStreamWarps * kStreamOutputs - 1) / (kStreamWarps * kStreamOutputs));
   EMBER_CHECK(grid.y <= 65535, "moe_down: %d outputs exceed one launch", width);

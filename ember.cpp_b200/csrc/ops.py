@@ -34,19 +34,22 @@ _SIGNATURES = {
     "ember_generalized_delta_rule": [_c_void, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_float,
                                      _c_float, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void,
                                      _c_int, _c_void],
-    "ember_moe_pick": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void, _c_void, _c_void],
+    "ember_moe_pick": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void, _c_void,
+                       _c_void],
+    "ember_moe_up": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                     _c_int, _c_void],
     "ember_post_norm": [_c_void, _c_float, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_float, _c_float,
                         _c_float, _c_void, _c_void, _c_void, _c_int, _c_void, _c_void, _c_int, _c_int, _c_void],
     "ember_depth_average": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_size, _c_void],
     "ember_qkv_prepare": [_c_void, ctypes.c_longlong, _c_void, ctypes.c_longlong, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
                           _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_float, _c_int,
-                          _c_void, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void],
+                          _c_void, _c_float, _c_int, _c_int, _c_void, ctypes.c_longlong, _c_int, _c_float, _c_int, _c_int, _c_void],
     "ember_poly_norm": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void],
     "ember_rglru": [_c_void, _c_void, _c_void, ctypes.c_longlong, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
                     _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
     "ember_rglru_step": [_c_void, _c_void, ctypes.c_longlong, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
                          _c_int, _c_int, _c_int, _c_void],
-    "ember_moe_combine": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_int, _c_int, _c_int, _c_void],
+    "ember_moe_combine": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void],
     "ember_moe_gate_up_act": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int,
                               _c_int, _c_int, _c_float, _c_float, _c_float, _c_void],
     "ember_conv_act": [_c_void, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void,
@@ -55,13 +58,13 @@ _SIGNATURES = {
                            _c_int, _c_int, _c_int, _c_void, _c_void, _c_float, _c_int, _c_int, _c_void],
     "ember_attention_plain_chunked": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int,
                                       _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void,
-                                      _c_int, _c_void],
+                                      _c_void, _c_int, _c_int, _c_void],
     "ember_attention_prefill_chunked": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
                                         _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void, _c_void,
-                                        _c_int, _c_void, _c_void],
+                                        _c_int, _c_void, _c_int, _c_void, _c_int, _c_void],
     "ember_attention_decode_chunked": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int,
                                        _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int,
-                                       _c_void, _c_void],
+                                       _c_void, _c_void, _c_int, _c_void],
     "ember_embed": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int, _c_float,
                     _c_void],
     "ember_layernorm": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_float, _c_int, _c_void],
@@ -122,16 +125,16 @@ _SIGNATURES = {
                              ctypes.c_longlong, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void],
     "ember_rotate": [_c_void, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void, ctypes.c_longlong, _c_int, _c_int, _c_int,
                      _c_int, _c_int, _c_int, _c_void, _c_void, _c_float, _c_int, _c_void],
-    "ember_latent_rows": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int, _c_float, _c_void, _c_float, _c_int,
+    "ember_latent_rows": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int, _c_float, _c_void, _c_float, _c_int, _c_int,
                           _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void],
     "ember_head_linear": [_c_void, ctypes.c_longlong, _c_int, _c_int, _c_void, _c_void, ctypes.c_longlong, _c_int, _c_int,
                           _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ember_head_linear_bf16": [_c_void, ctypes.c_longlong, _c_int, _c_void, _c_void, ctypes.c_longlong, _c_int, _c_int, _c_int,
                                _c_int, _c_int, _c_int, _c_void, _c_size, _c_void],
     "ember_latent_attention_plain": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int,
-                                     _c_int, _c_int, _c_int, _c_float, _c_int, _c_void],
+                                     _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void],
     "ember_latent_attention_mma": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int,
-                                   _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void],
+                                   _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_void],
     "ember_delta_rule": [_c_void, _c_void, ctypes.c_longlong, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void,
                          _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int,
                          _c_int, _c_void],
@@ -145,7 +148,7 @@ _SIGNATURES = {
     "ember_add_branches": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_float, _c_void],
     "ember_qkv_norm": [_c_void, ctypes.c_longlong, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int,
                        _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_void],
-    "ember_gate_mul": [_c_void, _c_void, ctypes.c_longlong, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
+    "ember_gate_mul": [_c_void, _c_void, ctypes.c_longlong, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ember_mlstm_gates": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void],
     "ember_mlstm_scan": [_c_void, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void,
                          _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void, _c_int, _c_void],
@@ -428,14 +431,14 @@ class CudaOps:
         return None
 
     def layernorm(self, x, w, b, eps, out_dtype):
-        """Layer norm of float32 rows."""
+        """Layer norm of float32 rows; b None: no bias."""
         rows, d = x.shape
-        if x.dtype != torch.float32 or w.dtype != torch.float32 or b.dtype != torch.float32:
+        if x.dtype != torch.float32 or any(t is not None and t.dtype != torch.float32 for t in (w, b)):
             raise KernelError("layernorm: input, gain and bias are float32")
-        if w.shape[0] != d or b.shape[0] != d:
-            raise KernelError(f"layernorm: width {d} with gain {tuple(w.shape)} and bias {tuple(b.shape)}")
+        if w.shape[0] != d or (b is not None and b.shape[0] != d):
+            raise KernelError(f"layernorm: width {d} with gain {tuple(w.shape)} and bias {None if b is None else tuple(b.shape)}")
         out = torch.empty((rows, d), dtype=out_dtype, device=x.device)
-        self._call("ember_layernorm", self._dense(x, "layernorm input").data_ptr(), w.data_ptr(), b.data_ptr(),
+        self._call("ember_layernorm", self._dense(x, "layernorm input").data_ptr(), w.data_ptr(), self._ptr(b),
                    out.data_ptr(), rows, d, float(eps), _code(out_dtype))
         return out
 
@@ -658,7 +661,7 @@ class CudaOps:
 
     def attention(self, qkv, cache, plan, n_heads, kv_heads, head_dim, scale, window, out_dtype, store=False,
                   keep_first=None, value_dim=None, slopes=None, sinks=None, chunk=0, head_scales=None,
-                  head_scales_positive=True):
+                  head_scales_positive=True, dist_bias=None):
         """Causal attention of the step's tokens over the cache.  With `store` their own keys and
         values are written into the cache first (in the same launch where a kernel can).
         float32: the plain kernel, whose sums depend on positions alone.  bfloat16: one token per
@@ -673,7 +676,8 @@ class CudaOps:
         chunk > 0 (in place of a window): a query at position p sees key j <= p only if floor(j / chunk) =
         floor(p / chunk).  head_scales (float32 per query head): one more factor on a head's scores; the
         tensor-core prompt kernel takes it where every factor is above zero (`head_scales_positive`).  Both go
-        the same way too."""
+        the same way too.  dist_bias (float32 [heads, n]): what a score gains after the scale by the distance to the key,
+        distances from n - 1 on taking the last column; the same way."""
         if qkv.dtype != cache.k.dtype or out_dtype != qkv.dtype:
             raise KernelError("attention: activations, cache and output have one element type")
         self._dense(qkv, "qkv")
@@ -682,10 +686,13 @@ class CudaOps:
                 raise KernelError(f"attention: {name} are float32 values, one a query head")
         if chunk < 0 or (chunk and (window or keep_first)):
             raise KernelError(f"attention: chunk {chunk} beside window {window} and {keep_first} kept positions")
-        if keep_first is not None or value_dim is not None or slopes is not None or sinks is not None or chunk or head_scales is not None:
+        if dist_bias is not None and (dist_bias.dtype != torch.float32 or dist_bias.dim() != 2 or dist_bias.shape[0] != n_heads
+                                      or not dist_bias.is_cuda or not dist_bias.is_contiguous()):
+            raise KernelError("attention: dist_bias is float32 [query heads, distances]")
+        if any(t is not None for t in (keep_first, value_dim, slopes, sinks, head_scales, dist_bias)) or chunk:
             return self._attention_kept(qkv, cache, plan, n_heads, kv_heads, head_dim, scale, window, out_dtype, store,
                                         int(keep_first or 0), head_dim if value_dim is None else int(value_dim), slopes, sinks,
-                                        int(chunk), head_scales, head_scales_positive)
+                                        int(chunk), head_scales, head_scales_positive, dist_bias)
         out = torch.empty((plan.T, n_heads * head_dim), dtype=out_dtype, device=qkv.device)
         pages = plan.pages[cache.group_index]
         if qkv.dtype == torch.bfloat16 and plan.all_single:
@@ -740,7 +747,8 @@ class CudaOps:
         return out
 
     def _attention_kept(self, qkv, cache, plan, n_heads, kv_heads, hd, scale, window, out_dtype, store, keep_first, vd,
-                        slopes=None, sinks=None, chunk=0, head_scales=None, head_scales_positive=True):
+                        slopes=None, sinks=None, chunk=0, head_scales=None, head_scales_positive=True, dist_bias=None):
+        n_dist = 0 if dist_bias is None else dist_bias.shape[1]
         if qkv.shape[1] != (n_heads + kv_heads) * hd + kv_heads * vd:
             raise KernelError(f"attention: rows of {qkv.shape[1]} values are not q | k | v of {n_heads} x {hd}, "
                               f"{kv_heads} x {hd} and {kv_heads} x {vd}")
@@ -762,22 +770,22 @@ class CudaOps:
                             out.data_ptr(), scratch.data_ptr(), plan.positions.data_ptr(), plan.seq_slot.data_ptr(),
                             pages.data_ptr(), plan.max_blocks, plan.T, n_heads, kv_heads, hd, vd, float(scale), int(window),
                             keep_first, int(max_keys), self._ptr(slopes), self._ptr(sinks), chunk, self._ptr(head_scales),
-                            allow=(2,))
+                            self._ptr(dist_bias), n_dist, allow=(2,))
             if rc == 0:
                 self.launches += 1      # (the merge)
                 return out
-        if fast and vd == hd and hd % 16 == 0 and hd <= 128 and scale > 0 and not plan.all_single and head_scales_positive:
+        if fast and vd % 16 == 0 and vd <= 128 and hd % 16 == 0 and hd <= 128 and scale > 0 and not plan.all_single and head_scales_positive:
             rc = self._call("ember_attention_prefill_chunked", qkv.data_ptr(), cache.k.data_ptr(), cache.v.data_ptr(),
                             out.data_ptr(), plan.seq_slot.data_ptr(), plan.seq_start.data_ptr(), plan.seq_new.data_ptr(),
                             plan.cu_new.data_ptr(), pages.data_ptr(), plan.max_blocks, plan.n, plan.max_new, n_heads,
                             kv_heads, hd, float(scale), int(window), keep_first, self._ptr(slopes), self._ptr(sinks), chunk,
-                            self._ptr(head_scales), allow=(2,))
+                            self._ptr(head_scales), vd, self._ptr(dist_bias), n_dist, allow=(2,))
             if rc == 0:
                 return out
         self._call("ember_attention_plain_chunked", qkv.data_ptr(), cache.k.data_ptr(), cache.v.data_ptr(), out.data_ptr(),
                    plan.positions.data_ptr(), plan.token_seq.data_ptr(), plan.seq_slot.data_ptr(), pages.data_ptr(),
                    plan.max_blocks, plan.T, n_heads, kv_heads, hd, float(scale), int(window), vd, keep_first,
-                   self._ptr(slopes), self._ptr(sinks), chunk, self._ptr(head_scales), _code(qkv.dtype))
+                   self._ptr(slopes), self._ptr(sinks), chunk, self._ptr(head_scales), self._ptr(dist_bias), n_dist, _code(qkv.dtype))
         return out
 
     # ------------------------------------------------------------------ branches side by side
@@ -979,15 +987,15 @@ class CudaOps:
                    int(temp_every), _code(proj.dtype), _code(out_dtype))
         return out
 
-    def gate_mul(self, a, proj, z_col, gate="sigmoid"):
-        """a * gate(z), z the columns from z_col of `proj`; gate "sigmoid" or "silu"."""
+    def gate_mul(self, a, proj, z_col, gate="sigmoid", span=1):
+        """a * gate(z), z the columns from z_col of `proj`, each for `span` neighbouring values of a; gate "sigmoid" or "silu"."""
         rows, n = a.shape
-        if gate not in ("silu", "sigmoid") or z_col + n > proj.shape[1] or proj.shape[0] != rows:
+        if gate not in ("silu", "sigmoid") or n % span or z_col + n // span > proj.shape[1] or proj.shape[0] != rows:
             raise KernelError("gate_mul: the gate's columns do not fit")
         out = torch.empty_like(a)
         z = proj[:, z_col:]
         self._call("ember_gate_mul", self._dense(a, "gated rows").data_ptr(), z.data_ptr(), proj.stride(0), out.data_ptr(), rows, n,
-                   1 if gate == "sigmoid" else 0, _code(a.dtype), _code(proj.dtype))
+                   1 if gate == "sigmoid" else 0, int(span), _code(a.dtype), _code(proj.dtype))
         return out
 
     # ------------------------------------------------------------------ mLSTM, minGRU
@@ -1107,7 +1115,7 @@ class CudaOps:
         return dst
 
     def latent_rows(self, down, plan, q_rank, q_norm, kv_norm, kv_rank, rot_dim, eps, rotary, cache, out_dtype):
-        """From float32 rows [T, q_rank (| kv_rank | rot_dim)]: the RMS-normed query row (returned, `out_dtype`), and with
+        """From float32 rows [T, q_rank (| kv_rank | rot_dim) (| others' columns)]: the RMS-normed query row (returned, `out_dtype`), and with
         a cache the RMS-normed row c and the rotated key part, written at each token's position into the cache's key
         and value pages."""
         T, width = down.shape
@@ -1122,7 +1130,7 @@ class CudaOps:
         pages = None if cache is None else plan.pages[cache.group_index]
         self._call("ember_latent_rows", self._dense(down, "rows").data_ptr(), width, int(q_rank), q_norm.data_ptr(),
                    self._ptr(kv_norm), int(kv_rank), int(rot_dim), float(eps), rotary.freqs.data_ptr(), float(rotary.magnitude),
-                   int(rotary.dims), c_q.data_ptr(), None if cache is None else cache.k.data_ptr(),
+                   int(rotary.dims), 1 if rotary.interleaved else 0, c_q.data_ptr(), None if cache is None else cache.k.data_ptr(),
                    None if cache is None else cache.v.data_ptr(), plan.positions.data_ptr(), plan.token_seq.data_ptr(),
                    plan.seq_slot.data_ptr(), self._ptr(pages), plan.max_blocks, T, _code(out_dtype))
         return c_q
@@ -1148,8 +1156,8 @@ class CudaOps:
                    out.data_ptr(), out.stride(0), int(out_col), int(out_head), T, heads, N, K, _code(w.dtype), _code(out.dtype))
         return out
 
-    def latent_attention(self, rows, cache, plan, heads, kv_rank, rot_dim, scale, out_dtype):
-        """Causal attention of the step's query heads (each `kv_rank` values for the cached rows, then `rot_dim` for the
+    def latent_attention(self, rows, cache, plan, heads, kv_rank, rot_dim, scale, out_dtype, window=0):
+        """Causal attention (over the last `window` positions, 0: all) of the step's query heads (each `kv_rank` values for the cached rows, then `rot_dim` for the
         shared key part) over the cache; per head the weighted sum of the cached rows: [T, heads * kv_rank]."""
         T = rows.shape[0]
         if rows.dtype != cache.k.dtype or out_dtype != rows.dtype or rows.shape[1] != heads * (kv_rank + rot_dim):
@@ -1161,6 +1169,8 @@ class CudaOps:
         if self.latent_fast and rows.dtype == torch.bfloat16:
             # one token each: the pages in chunks, a block a chunk, so that the launch fills the chip about twice
             blocks = min(plan.max_blocks, max(1, -(-plan.max_end // 64)))
+            if window > 0:                          # (the pages that the last `window` positions can touch)
+                blocks = min(blocks, (window + 62) // 64 + 1)
             n_chunks, per_chunk = 1, plan.max_blocks
             if plan.all_single and plan.T == plan.n:
                 tiles = plan.n * -(-heads // 64)
@@ -1172,14 +1182,15 @@ class CudaOps:
             rc = self._call("ember_latent_attention_mma", self._dense(rows, "query rows").data_ptr(), cache.k.data_ptr(),
                             cache.v.data_ptr(), out.data_ptr(), self._ptr(scratch), plan.seq_slot.data_ptr(),
                             plan.seq_start.data_ptr(), plan.cu_new.data_ptr(), pages.data_ptr(), plan.max_blocks, plan.n,
-                            max(int(plan.max_new), 1), T, heads, kv_rank, rot_dim, float(scale), n_chunks, per_chunk, allow=(2,))
+                            max(int(plan.max_new), 1), T, heads, kv_rank, rot_dim, float(scale), int(window), n_chunks, per_chunk,
+                            allow=(2,))
             if rc == 0:
                 self.launches += 1 if n_chunks > 1 else 0      # (the merge)
                 return out
         self._call("ember_latent_attention_plain", self._dense(rows, "query rows").data_ptr(), cache.k.data_ptr(),
                    cache.v.data_ptr(), out.data_ptr(), plan.positions.data_ptr(), plan.token_seq.data_ptr(),
                    plan.seq_slot.data_ptr(), pages.data_ptr(), plan.max_blocks, T, heads, kv_rank, rot_dim, float(scale),
-                   _code(rows.dtype))
+                   int(window), _code(rows.dtype))
         return out
 
     # ------------------------------------------------------------------ gated delta rule
@@ -1226,19 +1237,18 @@ class CudaOps:
                    _code(h.dtype))
         return out
 
-    def side_input(self, x, plan, table, col, dim, w_gate, w_proj, w_norm, eps):
+    def side_input(self, x, plan, table, col, dim, w_gate, w_proj, w_norm, eps, rows=None):
         """x += unit_rms(W_proj (gelu_tanh(W_gate x) * e)) * w_norm in place, e = `dim` columns from `col` of each token's
         row of `table`: the stream's rows in the compute type, the first product with its GELU, the table's values, the
-        second product with float32 sums, and the norm with the sum (`add_normed`)."""
+        second product with float32 sums, and the norm with the sum (`add_normed`).  rows: the stream's rows in the compute type,
+        where a launch in front left them."""
         T, width = x.shape
         dtype = w_gate.dtype
         if x.dtype != torch.float32 or table.dtype != dtype or w_proj.dtype != dtype or \
                 tuple(w_gate.shape) != (dim, width) or tuple(w_proj.shape) != (width, dim) or w_norm.numel() != width:
             raise KernelError("side_input: a float32 stream, the table and both matrices of one element type and fitting sizes")
-        rows = self._dense(x, "stream")
-        if dtype != torch.float32:
-            rows = torch.empty((T, width), dtype=dtype, device=x.device)
-            self._call("ember_cast_rows", x.data_ptr(), rows.data_ptr(), T * width, _code(dtype))
+        if rows is None:
+            rows = self.cast_rows(self._dense(x, "stream"), dtype)
         z = self.linear(rows, w_gate, None, act="gelu_tanh", out_dtype=dtype)
         g = torch.empty_like(z)
         self._call("ember_table_gate", z.data_ptr(), g.data_ptr(), plan.tokens.data_ptr(), table.data_ptr(), table.shape[0],
@@ -1324,32 +1334,49 @@ class CudaOps:
             tiled = dtype == torch.bfloat16 and pairs >= MOE_TILE_PAIRS
         return 1 if tiled and k % 8 == 0 and n_out % 2 == 0 else 0
 
-    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale, softmax=False):
+    _SCORES = {"sigmoid": 0, "softmax": 1, "softmax_all": 2}
+
+    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale, scores="sigmoid", group_top=2):
         """The router's choice for every row of float32 logits [T, >= experts]: scores sigmoid(z); chosen on score +
-        correction among the experts of the `keep_groups` groups (of `groups` equal groups of neighbours) whose two
-        largest choice scores add up to the most; weights = the chosen's scores over their sum (+ 1e-20) times
-        `route_scale`.  `softmax`: chosen on z + correction, weights = the softmax over the chosen's z + correction, times
-        `route_scale` (one group).  Returns (chosen int32 [T, top], weights float32 [T, top])."""
+        correction among the experts of the `keep_groups` groups (of `groups` equal groups of neighbours) whose
+        `group_top` (2 or 1) largest choice scores add up to the most; weights = the chosen's scores over their sum (+ 1e-20)
+        times `route_scale`.  scores "softmax": chosen on z + correction, weights = the softmax over the chosen's z + correction,
+        times `route_scale` (one group); "softmax_all": scores softmax(z), weights = the chosen's scores times `route_scale`.  Returns (chosen int32 [T, top], weights float32 [T, top])."""
         T = logits.shape[0]
         if logits.dtype != torch.float32 or logits.shape[1] < experts or correction.dtype != torch.float32 or correction.numel() != experts:
             raise KernelError("moe_pick: float32 logits of at least `experts` columns and a float32 correction an expert")
         chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
         weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
         self._call("ember_moe_pick", self._dense(logits, "logits").data_ptr(), logits.shape[1], correction.data_ptr(), T, int(experts),
-                   int(top), int(groups), int(keep_groups), float(route_scale), 1 if softmax else 0, chosen.data_ptr(), weights.data_ptr())
+                   int(top), int(groups), int(keep_groups), int(group_top), float(route_scale), self._SCORES[scores], chosen.data_ptr(),
+                   weights.data_ptr())
         return chosen, weights
 
-    def moe_combine(self, x, y, weights, shared, logits, gate_col):
+    def moe_combine(self, x, y, weights, shared, logits, gate_col, rows_dtype=None):
         """x + sum_k weights[:, k] * y[:, k, :] (+ shared, times sigmoid(logits[:, gate_col]) where logits are given),
-        float32, as a new tensor."""
+        float32, as a new tensor.  rows_dtype: returns (that, its rows in that type) from one launch."""
         T, top, width = y.shape
         if any(t is not None and t.dtype != torch.float32 for t in (x, y, weights, shared, logits)) or tuple(x.shape) != (T, width) \
                 or tuple(weights.shape) != (T, top) or (shared is not None and tuple(shared.shape) != (T, width)):
             raise KernelError("moe_combine: float32 rows of fitting sizes")
         out = torch.empty_like(x)
+        rows = torch.empty(x.shape, dtype=rows_dtype, device=x.device) if rows_dtype == torch.bfloat16 else None
         self._call("ember_moe_combine", self._dense(x, "stream").data_ptr(), self._dense(y, "experts' rows").data_ptr(),
                    self._dense(weights, "weights").data_ptr(), self._ptr(None if shared is None else self._dense(shared, "shared rows")),
-                   self._ptr(logits), 0 if logits is None else logits.shape[1], int(gate_col), out.data_ptr(), T, top, width)
+                   self._ptr(logits), 0 if logits is None else logits.shape[1], int(gate_col), out.data_ptr(), self._ptr(rows),
+                   T, top, width)
+        return out if rows_dtype is None else (out, out if rows is None else rows)
+
+    def moe_up(self, h, w_up, routing, out_dtype, act, tiled=None):
+        """The chosen experts' first product where an expert has no gate: act(W_up h) as [T * top, inner]."""
+        pair_expert, offsets, order, T, top, experts = routing
+        inner, width = w_up.shape[1], w_up.shape[2]
+        if h.dtype != w_up.dtype or out_dtype != h.dtype or h.shape[1] != width or w_up.shape[0] != experts or act not in _ACT:
+            raise KernelError("moe_up: rows, stacked matrices and output of one element type and fitting sizes")
+        out = torch.empty((T * top, inner), dtype=out_dtype, device=h.device)
+        self._call("ember_moe_up", self._dense(h, "rows").data_ptr(), self._dense(w_up, "experts").data_ptr(), pair_expert.data_ptr(),
+                   offsets.data_ptr(), order.data_ptr(), out.data_ptr(), T, top, experts, width, inner, _ACT[act],
+                   self._moe_tiled(T * top, h.dtype, tiled, width, inner), _code(h.dtype))
         return out
 
     def moe_gate_up(self, h, w_gate_up, routing, out_dtype, tiled=None, limit=0.0, alpha=1.0, shift=0.0):
@@ -1447,14 +1474,16 @@ class CudaOps:
     _QK_NORMS = {None: 0, "row": 1, "head": 2}
 
     def qkv_prepare(self, proj, plan, cache, heads, kv_heads, head_dim, value_dim, out_dtype, store, v_col=None, norm=None,
-                    q_gain=None, k_gain=None, eps=0.0, rotary=None, unit_after=False):
+                    q_gain=None, k_gain=None, eps=0.0, rotary=None, unit_after=False, mix=None, queries=True):
         """Norms, rotation and the cache's new rows in one launch, float32 in between: from rows q | k | v of `proj` (q alone
         where `store` is False: the keys and values are another layer's), the query heads into rows of q | k | v (the
         layout that `attention` reads; the rest of a row is not written) and the keys and values into the cache's
         pages.  norm "row": q and k divided by their root mean square over the whole row of heads and multiplied by gains of its
         width; "head": a head at a time, gains of the head's size (None: ones).  Then the rotation (a Rotary of
         parts/position.py, or None), then with `unit_after` every q and k head divided by its own root mean square.  v_col: the
-        column the values start at (default: behind the keys; the keys' own column makes them the keys as projected)."""
+        column the values start at (default: behind the keys; the keys' own column makes them the keys as projected).  mix = (rows [T, kv_heads x value_dim], lambda): the values become
+        (1 - lambda) * own + lambda * rows.  queries False: keys and values alone, for a `proj` that the attention reads
+        itself; returns None."""
         T = plan.T
         q_w, k_w = heads * head_dim, kv_heads * head_dim
         if norm not in self._QK_NORMS:
@@ -1467,15 +1496,21 @@ class CudaOps:
         if store and (cache.k.dtype != out_dtype or tuple(cache.k.shape[1:]) != (kv_heads, 64, head_dim)
                       or tuple(cache.v.shape[1:]) != (kv_heads, 64, value_dim)):
             raise KernelError("qkv_prepare: the cache's pages do not have the mixer's head sizes or element type")
-        out = torch.empty((T, q_w + k_w + kv_heads * value_dim), dtype=out_dtype, device=proj.device)
+        if not queries and (norm == "row" or not store):
+            raise KernelError("qkv_prepare: keys and values alone go into a cache and take no norm over rows")
+        other, blend = (None, 0.0) if mix is None else mix
+        if other is not None and (tuple(other.shape) != (T, kv_heads * value_dim) or other.stride(1) != 1 or not store):
+            raise KernelError("qkv_prepare: one row of values a token to blend in")
+        out = torch.empty((T, q_w + k_w + kv_heads * value_dim), dtype=out_dtype, device=proj.device) if queries else None
         pages = plan.pages[cache.group_index]
-        self._call("ember_qkv_prepare", proj.data_ptr(), proj.stride(0), out.data_ptr(), out.stride(0),
+        self._call("ember_qkv_prepare", proj.data_ptr(), proj.stride(0), self._ptr(out), out.stride(0) if queries else 0,
                    cache.k.data_ptr() if store else None, cache.v.data_ptr() if store else None, plan.positions.data_ptr(),
-                   plan.token_seq.data_ptr(), plan.seq_slot.data_ptr(), pages.data_ptr(), plan.max_blocks, T, heads,
+                   plan.token_seq.data_ptr(), plan.seq_slot.data_ptr(), pages.data_ptr(), plan.max_blocks, T, heads if queries else 0,
                    kv_heads if store else 0, head_dim, value_dim, q_w, q_w + k_w if v_col is None else int(v_col),
                    self._QK_NORMS[norm], self._ptr(q_gain), self._ptr(k_gain), float(eps), 1 if unit_after else 0,
                    None if rotary is None else rotary.freqs.data_ptr(), 1.0 if rotary is None else float(rotary.magnitude),
                    0 if rotary is None else int(rotary.dims), 1 if rotary is not None and rotary.interleaved else 0,
+                   self._ptr(other), 0 if other is None else other.stride(0), 0 if other is None else _code(other.dtype), float(blend),
                    _code(proj.dtype), _code(out_dtype))
         return out
 

@@ -5,7 +5,8 @@
 // through shared memory in float32, so that nothing is rounded between the norms and the rotation; the token's
 // angles are turned into cos and sin once for all heads.  Rounding to the compute type happens once, at the store.  Query
 // heads are written to the rows that the attention reads; keys and values go straight into the pages of the cache.
-// Values may be the keys as projected (before norm and rotation): v_col is then k_col.  A warp's sums depend on the
+// Values may be the keys as projected (before norm and rotation): v_col is then k_col.  With `blend` the values become
+// (1 - blend) * own + blend * another layer's of the same token.  Without query heads (heads 0) only keys and values are made.  A warp's sums depend on the
 // head's size alone, so a row's result does not depend on the batch.
 #include "common.cuh"
 
@@ -73,7 +74,22 @@ struct Prepare {
   int unit_after;                  // after the rotation: q and k heads divided by their root mean square
   int dims, interleaved;           // rotated dimensions of a head (0: none) and how they pair
   float magnitude, eps;
+  const void* other;               // the values that are blended in: kv_heads x vd a row, or null
+  long long other_stride;
+  int other_bf16;
+  float blend;
 };
+
+// W values of token t's row of the blended-in values, from column c on, folded into v
+template <int W>
+__device__ __forceinline__ void blend_values(const Prepare& a, int t, int c, float (&v)[W]) {
+  if (a.other == nullptr) return;
+  float o[W];
+  if (a.other_bf16) load_w<W>(static_cast<const __nv_bfloat16*>(a.other) + (size_t)t * a.other_stride + c, o);
+  else load_w<W>(static_cast<const float*>(a.other) + (size_t)t * a.other_stride + c, o);
+#pragma unroll
+  for (int e = 0; e < W; ++e) v[e] = (1.0f - a.blend) * v[e] + a.blend * o[e];
+}
 
 // W = 4: head sizes, columns and row strides are multiples of 4 and every pointer lies on 16 bytes (8 for bfloat16)
 template <typename TIN, typename TOUT, int W>
@@ -124,7 +140,7 @@ qkv_prepare_kernel(const TIN* __restrict__ in, long long in_stride, TOUT* __rest
   const int page = a.kv_heads > 0 ? pages[(size_t)s * max_blocks + p / kPage] : 0;
   const int total = a.heads + 2 * a.kv_heads;
   for (int it = blockIdx.y * kWarps + warp; it < total; it += gridDim.y * kWarps) {
-    if (it >= a.heads + a.kv_heads) {      // a value head: as projected
+    if (it >= a.heads + a.kv_heads) {      // a value head: as projected, or blended with another layer's
       if (page < 0) continue;
       const int g = it - a.heads - a.kv_heads;
       const TIN* src = row + a.v_col + (size_t)g * a.vd;
@@ -132,6 +148,7 @@ qkv_prepare_kernel(const TIN* __restrict__ in, long long in_stride, TOUT* __rest
       for (int i = lane * W; i < a.vd; i += 32 * W) {
         float v[W];
         load_w<W>(src + i, v);
+        blend_values<W>(a, t, g * a.vd + i, v);
         store_w<W>(dst + i, v);
       }
       continue;
@@ -282,7 +299,8 @@ qkv_prepare_short_kernel(const TIN* __restrict__ in, long long in_stride, TOUT* 
     for (int j = 0; j < kItems; ++j) {
       const int it = from + j * step;
       if (it >= total) break;
-      if (it >= n_qk) {      // a value head: as projected
+      if (it >= n_qk) {      // a value head: as projected, or blended with another layer's
+        if (col < a.vd) blend_values<4>(a, t, (it - n_qk) * a.vd + col, v[j]);
         if (page >= 0 && col < a.vd) store_w<4>(vc + (((size_t)page * a.kv_heads + it - n_qk) * kPage + place) * a.vd + col, v[j]);
         continue;
       }
@@ -339,13 +357,15 @@ qkv_prepare_short_kernel(const TIN* __restrict__ in, long long in_stride, TOUT* 
 
 // in [T, *]: q (heads x hd) from column 0, and with kv_heads > 0 k (kv_heads x hd) from k_col and v (kv_heads x vd) from
 // v_col.  out: rows of out_stride values whose first heads x hd are written.  kc, vc: the cache's pages (kv_heads > 0).
+// heads 0 (norm 0 or 2): keys and values alone, out is not touched.  other (float32 or bfloat16 rows of kv_heads x vd, or null):
+// the values become (1 - blend) * own + blend * other.
 // norm 0 none, 1 over the row (gains of the row's width), 2 a head at a time (gains of hd values); gains null: ones.
 EMBER_API int ember_qkv_prepare(const void* in, long long in_stride, void* out, long long out_stride, void* kc, void* vc,
                                 const int* positions, const int* token_seq, const int* seq_slot, const int* pages, int max_blocks,
                                 int T, int heads, int kv_heads, int hd, int vd, int k_col, int v_col, int norm, const float* q_gain,
                                 const float* k_gain, float eps, int unit_after, const float* freqs, float magnitude, int dims,
-                                int interleaved, int in_dtype, int out_dtype, cudaStream_t stream) {
-  EMBER_CHECK(T > 0 && heads > 0 && kv_heads >= 0 && hd > 0 && hd <= kMaxHead && vd > 0 && vd <= kMaxHead, "qkv_prepare: bad sizes");
+                                int interleaved, const void* other, long long other_stride, int other_dtype, float blend, int in_dtype, int out_dtype, cudaStream_t stream) {
+  EMBER_CHECK(T > 0 && heads >= 0 && kv_heads >= 0 && heads + kv_heads > 0 && (heads > 0 || norm != kNormRow) && hd > 0 && hd <= kMaxHead && vd > 0 && vd <= kMaxHead, "qkv_prepare: bad sizes");
   EMBER_CHECK(in_stride >= (long long)heads * hd && out_stride >= (long long)heads * hd, "qkv_prepare: rows too short for q");
   EMBER_CHECK(kv_heads == 0 || (k_col >= 0 && v_col >= 0 && in_stride >= (long long)k_col + (long long)kv_heads * hd &&
                                 in_stride >= (long long)v_col + (long long)kv_heads * vd && kc != nullptr && vc != nullptr &&
@@ -353,15 +373,19 @@ EMBER_API int ember_qkv_prepare(const void* in, long long in_stride, void* out, 
               "qkv_prepare: the keys' or values' columns do not fit the rows, or no cache");
   EMBER_CHECK(dims >= 0 && dims % 2 == 0 && dims <= hd && (dims == 0 || freqs != nullptr), "qkv_prepare: %d rotated dimensions of %d",
               dims, hd);
+  EMBER_CHECK(other == nullptr || (kv_heads > 0 && other_stride >= (long long)kv_heads * vd && (other_dtype == EMBER_F32 || other_dtype == EMBER_BF16)),
+              "qkv_prepare: the values to blend in do not fit");
   EMBER_CHECK(norm >= 0 && norm <= 2, "qkv_prepare: norm %d", norm);
   Prepare a;
   a.heads = heads, a.kv_heads = kv_heads, a.hd = hd, a.vd = vd, a.k_col = k_col, a.v_col = v_col, a.norm = norm;
   a.unit_after = unit_after, a.dims = dims, a.interleaved = interleaved, a.magnitude = magnitude, a.eps = eps;
+  a.other = other, a.other_stride = other_stride, a.other_bf16 = other_dtype == EMBER_BF16, a.blend = blend;
   const int total = heads + 2 * kv_heads;
   const int split = T >= 256 ? 1 : (total + kWarps - 1) / kWarps;      // few tokens: a warp a head over several blocks
   const dim3 grid(T, split < 65535 ? split : 65535);
   cudaError_t e;
   const bool vec = (hd | vd | k_col | v_col) % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 &&
+                   (other == nullptr || (other_stride % 4 == 0 && (uintptr_t)other % (other_dtype == EMBER_BF16 ? 8 : 16) == 0)) &&
                    ((uintptr_t)in | (uintptr_t)out | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)q_gain | (uintptr_t)k_gain) % 16 == 0;
   const bool brief = vec && hd <= 128 && vd <= 128;
 #define EMBER_PREP(TIN, TOUT)                                                                                                    \

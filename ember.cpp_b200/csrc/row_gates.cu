@@ -125,15 +125,65 @@ qkv_norm_kernel(const TIN* __restrict__ in, long long in_stride, TOUT* __restric
   }
 }
 
-// out = a * gate(z): kind 0 silu, 1 sigmoid.  z: n columns of a wider matrix.
-template <typename TA, typename TZ>
-__global__ void gate_mul_kernel(const TA* __restrict__ a, const TZ* __restrict__ z, long long z_stride, TA* __restrict__ out,
-                                size_t total, int n, int kind) {
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-    const size_t row = i / n;
-    const int c = (int)(i % n);
-    const float g = to_float(z[row * z_stride + c]);
-    out[i] = from_float<TA>(to_float(a[i]) * (kind == 1 ? sigmoidf(g) : g * sigmoidf(g)));
+// W values (4 or 1) from or to memory
+template <int W>
+__device__ __forceinline__ void load_w(const float* p, float (&v)[W]) {
+  if constexpr (W == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int W>
+__device__ __forceinline__ void load_w(const __nv_bfloat16* p, float (&v)[W]) {
+  if constexpr (W == 4) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    v[0] = lo.x, v[1] = lo.y, v[2] = hi.x, v[3] = hi.y;
+  } else {
+    v[0] = __bfloat162float(*p);
+  }
+}
+template <int W>
+__device__ __forceinline__ void store_w(float* p, const float (&v)[W]) {
+  if constexpr (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *p = v[0];
+}
+template <int W>
+__device__ __forceinline__ void store_w(__nv_bfloat16* p, const float (&v)[W]) {
+  if constexpr (W == 4) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    uint2 raw;
+    raw.x = *reinterpret_cast<const unsigned*>(&lo);
+    raw.y = *reinterpret_cast<const unsigned*>(&hi);
+    *reinterpret_cast<uint2*>(p) = raw;
+  } else {
+    *p = __float2bfloat16_rn(v[0]);
+  }
+}
+
+// out = a * gate(z): kind 0 silu, 1 sigmoid.  z: n / span columns of a wider matrix, each for `span` neighbouring values of
+// a.  grid (rows, blocks of columns).  W = 4: n and span (or, for span 1, z's rows) are whole fours on 16 bytes (8 in bfloat16).
+template <typename TA, typename TZ, int W>
+__global__ void __launch_bounds__(256)
+gate_mul_kernel(const TA* __restrict__ a, const TZ* __restrict__ z, long long z_stride, TA* __restrict__ out, int n, int kind, int span) {
+  const size_t row = blockIdx.x;
+  const TZ* zr = z + row * z_stride;
+  for (int c = (blockIdx.y * 256 + threadIdx.x) * W; c < n; c += gridDim.y * 256 * W) {
+    float v[W], g[W];
+    load_w<W>(a + row * n + c, v);
+    if (span == 1) {
+      load_w<W>(zr + c, g);
+    } else {
+      const float one = to_float(zr[c / span]);
+#pragma unroll
+      for (int e = 0; e < W; ++e) g[e] = one;
+    }
+#pragma unroll
+    for (int e = 0; e < W; ++e) v[e] *= kind == 1 ? sigmoidf(g[e]) : g[e] * sigmoidf(g[e]);
+    store_w<W>(out + row * n + c, v);
   }
 }
 
@@ -178,14 +228,21 @@ EMBER_API int ember_qkv_norm(const void* in, long long in_stride, void* out, con
   return 0;
 }
 
-EMBER_API int ember_gate_mul(const void* a, const void* z, long long z_stride, void* out, int rows, int n, int kind, int a_dtype,
-                             int z_dtype, cudaStream_t stream) {
-  EMBER_CHECK(rows > 0 && n > 0 && (kind == 0 || kind == 1) && z_stride >= n, "gate_mul: %d rows of %d, kind %d", rows, n, kind);
-  const size_t total = (size_t)rows * n;
-  const int grid = (int)((total + 255) / 256 < 65535 * 16 ? (total + 255) / 256 : 65535 * 16);
+EMBER_API int ember_gate_mul(const void* a, const void* z, long long z_stride, void* out, int rows, int n, int kind, int span,
+                             int a_dtype, int z_dtype, cudaStream_t stream) {
+  EMBER_CHECK(rows > 0 && n > 0 && (kind == 0 || kind == 1) && span >= 1 && n % span == 0 && z_stride >= n / span,
+              "gate_mul: %d rows of %d, kind %d, a gate for every %d values", rows, n, kind, span);
+  const uintptr_t a_bytes = a_dtype == EMBER_F32 ? 16 : 8, z_bytes = z_dtype == EMBER_F32 ? 16 : 8;
+  const bool four = n % 4 == 0 && ((uintptr_t)a | (uintptr_t)out) % a_bytes == 0 &&
+                    (span == 1 ? z_stride % 4 == 0 && (uintptr_t)z % z_bytes == 0 : span % 4 == 0);
+  const int w = four ? 4 : 1;
+  const dim3 grid(rows, (n + 256 * w - 1) / (256 * w) < 65535 ? (n + 256 * w - 1) / (256 * w) : 65535);
   cudaError_t e;
-#define EMBER_GM(TA, TZ) \
-  launch_plain(gate_mul_kernel<TA, TZ>, dim3(grid), dim3(256), 0, stream, (const TA*)a, (const TZ*)z, z_stride, (TA*)out, total, n, kind)
+#define EMBER_GM(TA, TZ)                                                                                                     \
+  (four ? launch_plain(gate_mul_kernel<TA, TZ, 4>, grid, dim3(256), 0, stream, (const TA*)a, (const TZ*)z, z_stride, (TA*)out, n, \
+                       kind, span)                                                                                           \
+        : launch_plain(gate_mul_kernel<TA, TZ, 1>, grid, dim3(256), 0, stream, (const TA*)a, (const TZ*)z, z_stride, (TA*)out, n, \
+                       kind, span))
   if (a_dtype == EMBER_F32 && z_dtype == EMBER_F32) e = EMBER_GM(float, float);
   else if (a_dtype == EMBER_BF16 && z_dtype == EMBER_F32) e = EMBER_GM(__nv_bfloat16, float);
   else if (a_dtype == EMBER_BF16 && z_dtype == EMBER_BF16) e = EMBER_GM(__nv_bfloat16, __nv_bfloat16);

@@ -82,6 +82,8 @@ class StepContext:
     next_weights: tuple = ()   # set by the model: the first matrix that the block after the current one streams
     model_state: dict = dataclasses.field(default_factory=dict)   # per-sequence state of the parts in front of the layers
     history: list = dataclasses.field(default_factory=list)       # results of the layers so far, where a layer sums over them
+    kept: dict = dataclasses.field(default_factory=dict)          # what a layer leaves for later layers of the step, by name
+    rows_wanted: bool = False                                     # the stream's rows in the compute type are read next
     noted: tuple = (None, None)                                   # a float32 stream and its rows in the compute type
 
     def note_rows(self, stream, rows) -> None:

@@ -43,6 +43,14 @@ projected (biases included), before norm and rotation, and there is no value mat
 tensors of keys and values and reads the keys and values that another entry of the schedule cached.  With any of these,
 or with both norms and a rotation, the projection stays in float32 and one launch makes norms and rotation of q and
 k, rounds once, and puts keys and values straight into the cache's pages (`ops.qkv_prepare`).
+
+And: `out_bias` = suffix: the output projection has a bias of that suffix; `gate_scope` = "head": the gate's matrix has one
+row a head and the whole head's output is multiplied by its sigmoid (also beside convolutions); `distance_bias` = (name,
+far, rows): a table [rows, heads] whose entry for the bucket of the distance to the key (`position.distance_buckets`) is
+added to a score after the scale (`rows` is what random-weights mode draws; a checkpoint's table has its own number);
+`value_mix`: "keep" leaves the layer's values (after the convolution, before the cache) for later layers of the step, any
+other name is that of a stored number lambda, and the values become (1 - lambda) * own + lambda * those kept, before they are
+cached (values carried from the first layer: Zhou et al., "Value Residual Learning").
 """
 from __future__ import annotations
 
@@ -62,7 +70,8 @@ class CausalAttention(Mixer):
                  value_norm: bool = False, norm_eps: float = 0.0, q_temp=None, distance_slope_base: float | None = None,
                  sink: str | None = None, gate: str | None = None, qkv_bias: str | None = None, conv=None, rotary=None,
                  head_scale: str | None = None, chunk: int = 0, fixed_sink: float | None = None, qk_norm_scope: str = "row",
-                 unit_qk: bool = False, values_are_keys: bool = False, shares_cache: bool = False):
+                 unit_qk: bool = False, values_are_keys: bool = False, shares_cache: bool = False, out_bias: str | None = None,
+                 gate_scope: str = "value", distance_bias=None, value_mix: str | None = None):
         super().__init__(prefix)
         if n_heads % kv_heads:
             raise ValueError(f"attention {prefix!r}: {n_heads} heads are not a multiple of {kv_heads} key/value heads")
@@ -81,8 +90,21 @@ class CausalAttention(Mixer):
         self.slope_base = None if distance_slope_base is None else float(distance_slope_base)
         self.sink_name = None if sink is None else prefix + sink
         self.gate_name = None if gate is None else prefix + gate
+        if gate_scope not in ("value", "head"):
+            raise ValueError(f"attention {prefix!r}: gate_scope = {gate_scope!r}")
+        self.gate_scope = gate_scope
         # rows that pass a norm, a temperature or a gate between the projection and the attention
-        self.prepared = self.qk_norm_names is not None or self.value_norm or self.q_temp is not None or self.gate_name is not None
+        self.prepared = (self.qk_norm_names is not None or self.value_norm or self.q_temp is not None
+                         or (self.gate_name is not None and conv is None))
+        self.out_bias_name = None if out_bias is None else prefix + out + out_bias
+        if out_bias is not None and bias:
+            raise ValueError(f"attention {prefix!r}: an output bias by its suffix comes without the fused projection's biases")
+        self.distance_bias = None
+        if distance_bias is not None:
+            self.distance_bias = (prefix + distance_bias[0], float(distance_bias[1]), int(distance_bias[2]))
+        self.value_mix = value_mix
+        self.value_lambda_name = None if value_mix in (None, "keep") else prefix + value_mix
+        self.value_lambda = 0.0
         self.fixed_sink = None if fixed_sink is None else float(fixed_sink)
         self.chunk = int(chunk)
         self.head_scale_name = None if head_scale is None else prefix + head_scale
@@ -117,8 +139,13 @@ class CausalAttention(Mixer):
                              "cache come with q, k and v stored apart, without value norms, temperatures, gates or convolutions")
         if self.values_are_keys and value_dim is not None and int(value_dim) != int(head_dim):
             raise ValueError(f"attention {prefix!r}: values that are the keys have the keys' size, not {value_dim}")
+        if value_mix is not None and (self.shares_cache or self.values_are_keys or not (self.one_prepare or conv is not None)):
+            raise ValueError(f"attention {prefix!r}: values that are kept or blended come with values of the layer's own, after norms "
+                             "a head or convolutions")
+        if conv is not None and (qk_norm is not None or value_norm or q_temp is not None):
+            raise ValueError(f"attention {prefix!r}: convolutions come without norms and temperatures")
         self.biased = (self.slope_base is not None or self.sink_name is not None or self.fixed_sink is not None
-                       or self.chunk > 0 or self.head_scale_name is not None)
+                       or self.chunk > 0 or self.head_scale_name is not None or distance_bias is not None)
         if (self.prepared or self.one_prepare or slope_base_or_sink(distance_slope_base, sink)) and bias:
             raise ValueError(f"attention {prefix!r}: norms, gates, slopes and sinks come without biases")
         self.extended = int(keep_first) > 0 or value_dim is not None or self.prepared or self.biased or self.one_prepare
@@ -138,7 +165,7 @@ class CausalAttention(Mixer):
         self.widths = (self.q_width, self.kv_heads * self.head_dim, self.kv_heads * self.value_dim)
         self.qkv_width = sum(self.widths)
         self.w_qkv = self.b_qkv = self.w_out = self.b_out = None
-        self.q_gain = self.k_gain = self.sinks = self.slopes = None
+        self.q_gain = self.k_gain = self.sinks = self.slopes = self.dist_bias = None
 
     def _shape(self, n_in, n_out):
         return (n_in, n_out) if self.stored == "in_out" else (n_out, n_in)
@@ -164,7 +191,14 @@ class CausalAttention(Mixer):
         if self.sink_name is not None:
             specs.append(WeightSpec(self.sink_name, (self.n_heads,), std=1.0))
         if self.gate_name is not None:
-            specs.append(WeightSpec(self.gate_name + self.suffix, self._shape(self.width, self.o_width), std=self.init_std))
+            n = self.n_heads if self.gate_scope == "head" else self.o_width
+            specs.append(WeightSpec(self.gate_name + self.suffix, self._shape(self.width, n), std=self.init_std))
+        if self.out_bias_name is not None:
+            specs.append(WeightSpec(self.out_bias_name, (self.width,), std=self.bias_init_std))
+        if self.distance_bias is not None:
+            specs.append(WeightSpec(self.distance_bias[0], (self.distance_bias[2], self.n_heads), std=1.0, free=(0,)))
+        if self.value_lambda_name is not None:
+            specs.append(WeightSpec(self.value_lambda_name, (), mean=0.5, std=0.1))
         if self.qkv_bias_suffix is not None:
             specs += [WeightSpec(n + self.qkv_bias_suffix, (w,), std=self.bias_init_std * 10) for n, w in self._projections()]
         if self.conv is not None:
@@ -201,6 +235,16 @@ class CausalAttention(Mixer):
         if self.bias:
             self.b_qkv = runtime.vector(get(self.qkv_name + ".bias"))
             self.b_out = runtime.vector(get(self.out_name + ".bias"))
+        if self.out_bias_name is not None:
+            self.b_out = runtime.vector(get(self.out_bias_name))
+        if self.distance_bias is not None:      # spread over the distances: [heads, distances], the last column for all beyond
+            from .position import distance_buckets
+            table = runtime.vector(get(self.distance_bias[0]))
+            of = distance_buckets(table.shape[0], self.distance_bias[1])
+            of = of[:max(1, min(len(of), self.chunk or self.window or len(of)))]
+            self.dist_bias = table[torch.tensor(of, device=table.device)].t().contiguous()
+        if self.value_lambda_name is not None:
+            self.value_lambda = float(get(self.value_lambda_name))
         if self.qkv_bias_suffix is not None:
             self.b_qkv = torch.cat([runtime.vector(get(n + self.qkv_bias_suffix)) for n, _ in self._projections()]).contiguous()
         if self.conv is not None:
@@ -243,15 +287,33 @@ class CausalAttention(Mixer):
         norm = None if self.qk_norm_names is None else self.qk_norm_scope
         qkv = ops.qkv_prepare(proj, ctx.plan, app.cache, self.n_heads, self.kv_heads, self.head_dim, self.value_dim, ctx.dtype,
                               store=not self.shares_cache, v_col=self.q_width if self.values_are_keys else None, norm=norm,
-                              q_gain=self.q_gain, k_gain=self.k_gain, eps=self.norm_eps, rotary=self.rotary, unit_after=self.unit_qk)
-        more = dict(slopes=self.slopes, sinks=self.sinks, chunk=self.chunk, head_scales=self.head_scales,
-                    head_scales_positive=self.head_scales is None or self.head_scales_positive)
+                              q_gain=self.q_gain, k_gain=self.k_gain, eps=self.norm_eps, rotary=self.rotary, unit_after=self.unit_qk,
+                              **self._value_mix(ctx, proj))
+        more = self._sight()
         if self._plain_sight():
             return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
                                  out_dtype=ctx.dtype, store=False)
         return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
                              out_dtype=ctx.dtype, store=False, keep_first=self.keep_first if self.window > 0 else 0,
                              value_dim=self.value_dim, **more)
+
+    def _sight(self) -> dict:
+        """What the attention's kernels take beside heads, scale and window."""
+        more = dict(slopes=self.slopes, sinks=self.sinks, chunk=self.chunk, head_scales=self.head_scales,
+                    head_scales_positive=self.head_scales is None or self.head_scales_positive)
+        if self.dist_bias is not None:
+            more["dist_bias"] = self.dist_bias
+        return more
+
+    def _value_mix(self, ctx, rows) -> dict:
+        """`rows` [T, q | k | v ...]: keeps the columns of the values for later layers of the step, or names those kept and
+        their weight in the blend."""
+        if self.value_mix is None:
+            return {}
+        if self.value_mix == "keep":
+            ctx.kept["values"] = rows[:, sum(self.widths[:2]):self.qkv_width]
+            return {}
+        return {"mix": (ctx.kept["values"], self.value_lambda)}
 
     def _plain_sight(self) -> bool:
         """Nothing but a window on the scores, and the head size at which the kernels for such heads are the faster ones (one
@@ -274,26 +336,30 @@ class CausalAttention(Mixer):
             o = ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
                               out_dtype=ctx.dtype, store=app.writes_cache, keep_first=self.keep_first if self.window > 0 else 0,
                               value_dim=self.value_dim, slopes=self.slopes, sinks=self.sinks)
-            return o if self.gate_name is None else ops.gate_mul(o, proj, self.gate_col, "sigmoid")
-        qkv = ops.linear(h, self.w_qkv, self.b_qkv, out_dtype=ctx.dtype)
+            return o if self.gate_name is None else self._gated(ctx, o, proj)
+        qkv = proj = ops.linear(h, self.w_qkv, self.b_qkv, out_dtype=ctx.dtype)
+        store = app.writes_cache
         if self.conv is not None:
             state = app.state.get("conv") if isinstance(app.state, dict) else None
             qkv = ops.conv_silu(qkv, 0, self.qkv_width, self.conv_w, self.conv_b, state, ctx.plan, act="none")
         ctx.position.apply_qk(ctx, qkv, self.n_heads, self.kv_heads, self.head_dim)
         if self.rotary is not None:
             self.rotary.apply_qk(ctx, qkv, self.n_heads, self.kv_heads, self.head_dim)
-        if self.chunk > 0 or self.head_scales is not None:
-            return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale,
-                                 self.window, out_dtype=ctx.dtype, store=app.writes_cache, keep_first=0, value_dim=self.value_dim,
-                                 slopes=self.slopes, sinks=self.sinks, chunk=self.chunk, head_scales=self.head_scales,
-                                 head_scales_positive=self.head_scales is None or self.head_scales_positive)
+        if self.value_mix is not None:      # the keys and the blended values go into the cache by a launch of their own
+            ops.qkv_prepare(qkv, ctx.plan, app.cache, self.n_heads, self.kv_heads, self.head_dim, self.value_dim, ctx.dtype,
+                            store=True, queries=False, **self._value_mix(ctx, qkv))
+            store = False
         if not self.extended:
-            return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale,
-                                 self.window, out_dtype=ctx.dtype, store=app.writes_cache)
-        return ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale,
-                             self.window, out_dtype=ctx.dtype, store=app.writes_cache,
-                             keep_first=self.keep_first if self.window > 0 else 0, value_dim=self.value_dim,
-                             slopes=self.slopes, sinks=self.sinks)
+            o = ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale,
+                              self.window, out_dtype=ctx.dtype, store=store)
+        else:
+            o = ops.attention(qkv, app.cache, ctx.plan, self.n_heads, self.kv_heads, self.head_dim, self.scale, self.window,
+                              out_dtype=ctx.dtype, store=store, keep_first=self.keep_first if self.window > 0 else 0,
+                              value_dim=self.value_dim, **self._sight())
+        return o if self.gate_name is None else self._gated(ctx, o, proj)
+
+    def _gated(self, ctx, o, proj):
+        return ctx.ops.gate_mul(o, proj, self.gate_col, "sigmoid", **({"span": self.value_dim} if self.gate_scope == "head" else {}))
 
     def forward(self, ctx, h, residual, app):
         return ctx.ops.linear(self._attend(ctx, h, app), self.w_out, self.b_out, residual=residual)

@@ -44,7 +44,9 @@ class PreNormBlock(Block):
         x = self.mixer.forward(ctx, h, x, app)
         if self.ffn is not None:
             h = self.norm2.forward(ctx, x, ctx.dtype)
+            ctx.rows_wanted = bool(self.addons)     # what follows reads the stream's rows in the compute type
             x = self.ffn.forward(ctx, h, x)
+            ctx.rows_wanted = False
         return self.add_ons(ctx, x)
 
 

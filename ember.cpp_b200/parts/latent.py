@@ -15,6 +15,10 @@ query is carried into the row's space (one small product per head), the attentio
 k_r directly with all heads sharing the cached rows, its output is a weighted sum of rows c per
 head, and W_uv[h] expands that sum (one small product per head) before the output projection.
 
+With `window` > 0 a query at position p sees the cached rows of positions p - window + 1 .. p, and the cache keeps those
+alone.  `gate` names a matrix W_g: the heads' outputs laid end to end are multiplied by sigmoid(W_g h), value by value,
+before the output projection; its rows join the down projections, which stay one product.
+
 A layer with `shares_cache` has no W_dkv: its schedule entry names the entry whose cached rows it
 reads (`Application.cache_of`), with its own queries, W_uk, W_uv and output projection.
 """
@@ -29,8 +33,11 @@ class LatentAttention(Mixer):
     def __init__(self, prefix: str, width: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int,
                  scale: float, eps: float, rotary: dict, shares_cache: bool = False, dq: str = "dq", uq: str = "uq",
                  dkv: str = "dkv", uk: str = "uk", uv: str = "uv", out: str = "o", norm_suffix: str = ".norm",
-                 init_std: float = 0.02, out_init_std: float = 0.02):
+                 init_std: float = 0.02, out_init_std: float = 0.02, window: int = 0, gate: str | None = None):
         super().__init__(prefix)
+        self.window, self.gate_name = int(window), None if gate is None else prefix + gate
+        if self.window < 0:
+            raise ValueError(f"latent attention {prefix!r}: window {self.window}")
         self.width, self.heads, self.dim, self.rot_dim, self.vdim = int(width), int(heads), int(dim), int(rot_dim), int(vdim)
         self.q_rank, self.kv_rank, self.scale, self.eps = int(q_rank), int(kv_rank), float(scale), float(eps)
         self.shares_cache = bool(shares_cache)
@@ -55,6 +62,8 @@ class LatentAttention(Mixer):
         if not self.shares_cache:
             specs += [WeightSpec(n["dkv"], (self.row, d), std=self.init_std),
                       WeightSpec(n["dkv"] + self.norm_suffix, (self.kv_rank,), mean=1.0, std=0.1)]
+        if self.gate_name is not None:
+            specs.append(WeightSpec(self.gate_name, (self.heads * self.vdim, d), std=self.init_std))
         return specs + [WeightSpec(n["uk"], (self.heads * self.dim, self.kv_rank), std=self.init_std),
                         WeightSpec(n["uv"], (self.heads * self.vdim, self.kv_rank), std=self.init_std),
                         WeightSpec(n["out"], (d, self.heads * self.vdim), std=self.out_init_std)]
@@ -63,7 +72,12 @@ class LatentAttention(Mixer):
         import torch
         n = self.names
         down = [runtime.matrix(get(n["dq"]))] + ([] if self.shares_cache else [runtime.matrix(get(n["dkv"]))])
-        self.w_down = torch.cat(down).contiguous()            # one product for both down projections
+        if self.gate_name is not None:                        # the gate's rows behind them, from a multiple of 8 columns on
+            used = sum(w.shape[0] for w in down)
+            self.gate_col = -(-used // 8) * 8
+            down.append(torch.zeros((self.gate_col - used, self.width), dtype=down[0].dtype, device=down[0].device))
+            down.append(runtime.matrix(get(self.gate_name)))
+        self.w_down = torch.cat(down).contiguous()            # one product for the down projections (and the gate)
         self.q_norm = runtime.vector(get(n["dq"] + self.norm_suffix))
         self.kv_norm = None if self.shares_cache else runtime.vector(get(n["dkv"] + self.norm_suffix))
         self.w_uq = runtime.matrix(get(n["uq"]))
@@ -78,7 +92,7 @@ class LatentAttention(Mixer):
         return [self.w_down, self.w_uq, self.w_out]
 
     def cache_need(self):
-        return CacheNeed("full", 1, self.kv_rank, 0, 0, self.rot_dim)
+        return CacheNeed("window" if self.window > 0 else "full", 1, self.kv_rank, self.window, 0, self.rot_dim)
 
     def _attend(self, ctx, h, app):
         import torch
@@ -86,7 +100,7 @@ class LatentAttention(Mixer):
         if app.writes_cache == self.shares_cache:
             raise ValueError(f"latent attention {self.prefix!r}: a layer with a down projection of its own writes the "
                              "cache, a layer without one reads another entry's")
-        down = ops.linear(h, self.w_down, None, out_dtype=torch.float32)             # [T, q_rank (| kv_rank | rot_dim)]
+        down = ops.linear(h, self.w_down, None, out_dtype=torch.float32)             # [T, q_rank (| kv_rank | rot_dim) (| gate)]
         # the two norms, the shared key part's rotation and the write of c and k_r into the cache in one launch
         c_q = ops.latent_rows(down, ctx.plan, self.q_rank, self.q_norm, self.kv_norm, self.kv_rank, self.rot_dim, self.eps,
                               self.rotary, app.cache if app.writes_cache else None, ctx.dtype)
@@ -94,9 +108,11 @@ class LatentAttention(Mixer):
         rows = torch.empty((q.shape[0], self.heads * self.row), dtype=ctx.dtype, device=q.device)
         ops.head_linear(q, 0, self.q_head, self.w_uk_t, rows, 0, self.row)           # the plain parts, carried over
         self.rotary.rotate(ctx, q, rows, self.heads, self.dim, self.q_head, self.kv_rank, self.row, self.rot_dim)
-        mixed = ops.latent_attention(rows, app.cache, ctx.plan, self.heads, self.kv_rank, self.rot_dim, self.scale, ctx.dtype)
+        mixed = ops.latent_attention(rows, app.cache, ctx.plan, self.heads, self.kv_rank, self.rot_dim, self.scale, ctx.dtype,
+                                     **({"window": self.window} if self.window > 0 else {}))
         out = torch.empty((q.shape[0], self.heads * self.vdim), dtype=ctx.dtype, device=q.device)
-        return ops.head_linear(mixed, 0, self.kv_rank, self.w_uv, out, 0, self.vdim)
+        ops.head_linear(mixed, 0, self.kv_rank, self.w_uv, out, 0, self.vdim)
+        return out if self.gate_name is None else ops.gate_mul(out, down, self.gate_col, "sigmoid")
 
     def forward(self, ctx, h, residual, app):
         return ctx.ops.linear(self._attend(ctx, h, app), self.w_out, None, residual=residual)

@@ -94,7 +94,11 @@ class RoutedExperts(FeedForward):
     An optional shared expert of the same form (sizes and limit of its own) runs for every token and is added,
     multiplied by sigmoid(w_sg . h), one number a token, where `shared_gate` names w_sg.
     With `scores` "softmax" the stored vector is a bias of the logits: the `top` largest of z + bias are chosen and weigh
-    the softmax over the chosen ones alone (times `route_scale`); experts are then in one group.
+    the softmax over the chosen ones alone (times `route_scale`); experts are then in one group.  With `scores` "softmax_all"
+    the scores are the softmax over all experts, the choice is made on score + correction and the chosen's scores weigh as
+    they are (times `route_scale`).  `group_top`: how many of a group's largest choice scores make its score (2, or 1).
+    `gate` None: an expert has no gate, `down(act(up h))` with `activation` "relu2" (the square of relu), and so has the
+    shared one.
 
     The router's rows and the shared expert's gate row are one product with float32 sums; scores, choice,
     weights and the weighted sum are float32.  Nothing returns to the host."""
@@ -103,10 +107,13 @@ class RoutedExperts(FeedForward):
                  groups: int = 1, keep_groups: int = 1, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
                  shared_inner: int = 0, shared_limit: float = 0.0, shared_gate: str | None = None,
                  scores: str = "sigmoid", router: str = "router", correction: str | None = "correction", expert: str = "e{}.", shared: str = "shared.",
-                 gate: str = "gate", up: str = "up", down: str = "down", suffix: str = "", init_std: float = 0.02,
-                 down_init_std: float = 0.02):
+                 gate: str | None = "gate", up: str = "up", down: str = "down", suffix: str = "", init_std: float = 0.02,
+                 down_init_std: float = 0.02, group_top: int = 2, activation: str = "relu2"):
         super().__init__(prefix)
         self.width, self.experts, self.top, self.inner = int(width), int(experts), int(top), int(inner)
+        self.group_top, self.gated, self.activation = int(group_top), gate is not None, str(activation)
+        if self.group_top not in (1, 2) or (not self.gated and (activation != "relu2" or limit or shared_gate is not None)):
+            raise ValueError(f"experts {prefix!r}: group_top = {group_top}, and without a gate {activation!r} with limit {limit}")
         self.groups, self.keep_groups, self.route_scale = int(groups), int(keep_groups), float(route_scale)
         self.limit, self.alpha, self.shift = float(limit), float(alpha), float(shift)
         if not 1 <= self.top <= self.experts or self.top > 32 or self.experts > 1024:
@@ -116,15 +123,20 @@ class RoutedExperts(FeedForward):
         if self.keep_groups * (self.experts // self.groups) < self.top:
             raise ValueError(f"experts {prefix!r}: {self.keep_groups} groups of {self.experts // self.groups} hold fewer "
                              f"than top = {self.top} experts")
-        if scores not in ("sigmoid", "softmax") or (scores == "softmax" and self.groups != 1):
+        if scores not in ("sigmoid", "softmax", "softmax_all") or (scores == "softmax" and self.groups != 1):
             raise ValueError(f"experts {prefix!r}: scores = {scores!r} with {self.groups} groups")
-        self.softmax = scores == "softmax"
+        self.scores = scores
         self.router_name = prefix + router
         self.correction_name = None if correction is None else prefix + correction
-        self.expert_names = [tuple(prefix + expert.format(e) + n + suffix for n in (gate, up, down)) for e in range(self.experts)]
+        self.expert_names = [tuple(prefix + expert.format(e) + n + suffix for n in ((gate, up, down) if self.gated else (up, down)))
+                             for e in range(self.experts)]
         self.init_std, self.down_init_std = init_std, down_init_std
         self.shared = self.shared_gate_name = None
-        if shared_inner:
+        if shared_inner and not self.gated:
+            self.shared = build_part("ffn", PartSpec("dense", prefix + shared, dict(
+                width=width, inner=int(shared_inner), activation=activation, up=up, down=down, stored="out_in", bias=False,
+                suffix=suffix, any_size=True, init_std=init_std, down_init_std=down_init_std)))
+        elif shared_inner:
             act = dict(activation="clamped_sigmoid", limit=float(shared_limit), alpha=alpha, shift=shift) if shared_limit > 0 \
                 else dict(activation="silu")
             self.shared = build_part("ffn", PartSpec("gated", prefix + shared, dict(
@@ -137,10 +149,9 @@ class RoutedExperts(FeedForward):
         specs = [WeightSpec(self.router_name, (self.experts, self.width), std=0.3)]
         if self.correction_name is not None:
             specs.append(WeightSpec(self.correction_name, (self.experts,), std=0.1))
-        for g, u, d in self.expert_names:
-            specs += [WeightSpec(g, (self.inner, self.width), std=self.init_std),
-                      WeightSpec(u, (self.inner, self.width), std=self.init_std),
-                      WeightSpec(d, (self.width, self.inner), std=self.down_init_std)]
+        for *into, d in self.expert_names:
+            specs += [WeightSpec(n, (self.inner, self.width), std=self.init_std) for n in into]
+            specs.append(WeightSpec(d, (self.width, self.inner), std=self.down_init_std))
         if self.shared is not None:
             specs += self.shared.weight_specs()
             if self.shared_gate_name is not None:
@@ -159,8 +170,9 @@ class RoutedExperts(FeedForward):
         self.w_router = w.contiguous()
         self.correction = (torch.zeros(self.experts, dtype=torch.float32, device=w.device) if self.correction_name is None
                            else runtime.vector(get(self.correction_name)))
-        self.w_gate_up = torch.stack([torch.cat([runtime.matrix(get(g)), runtime.matrix(get(u))]) for g, u, _ in self.expert_names]).contiguous()
-        self.w_down = torch.stack([runtime.matrix(get(d)) for _, _, d in self.expert_names]).contiguous()
+        # [experts, gate | up, width], or without a gate [experts, up, width]
+        self.w_gate_up = torch.stack([torch.cat([runtime.matrix(get(n)) for n in into]) for *into, _ in self.expert_names]).contiguous()
+        self.w_down = torch.stack([runtime.matrix(get(names[-1])) for names in self.expert_names]).contiguous()
         if self.shared is not None:
             self.shared.load(get, runtime)
 
@@ -170,10 +182,13 @@ class RoutedExperts(FeedForward):
     def _chosen(self, ctx, h, logits):
         ops = ctx.ops
         chosen, weights = ops.moe_pick(logits, self.correction, self.experts, self.top, self.groups, self.keep_groups,
-                                       self.route_scale, **({"softmax": True} if self.softmax else {}))
+                                       self.route_scale, scores=self.scores, group_top=self.group_top)
         routing = ops.moe_route(None, ctx.plan.T, chosen, self.experts, self.top)
-        inner = ops.moe_gate_up(h, self.w_gate_up, routing, out_dtype=ctx.dtype, limit=self.limit, alpha=self.alpha,
-                                shift=self.shift)                                     # [T * top, inner]
+        if self.gated:
+            inner = ops.moe_gate_up(h, self.w_gate_up, routing, out_dtype=ctx.dtype, limit=self.limit, alpha=self.alpha,
+                                    shift=self.shift)                                 # [T * top, inner]
+        else:
+            inner = ops.moe_up(h, self.w_gate_up, routing, out_dtype=ctx.dtype, act=self.activation)
         return ops.moe_down(inner, self.w_down, routing), weights                     # float32 [T, top, width], [T, top]
 
     def forward(self, ctx, h, residual):
@@ -181,12 +196,19 @@ class RoutedExperts(FeedForward):
         logits = ctx.ops.linear(h, self.w_router, None, out_dtype=torch.float32)      # float32 [T, experts (| sg) (| 0)]
         if self.shared is None:
             y, weights = self._chosen(ctx, h, logits)
-            return ctx.ops.moe_combine(residual, y, weights, None, None, 0)
+            return self._combined(ctx, residual, y, weights, None, None)
         runs = [lambda: self._chosen(ctx, h, logits), lambda: self.shared.branches(ctx, h)[0][0]]
         together = getattr(ctx.ops, "side_by_side", None)     # (one-token steps: the shared expert beside the chosen ones)
         (y, weights), shared = together(runs) if together is not None and ctx.plan.all_single else [run() for run in runs]
-        gated = self.shared_gate_name is not None
-        return ctx.ops.moe_combine(residual, y, weights, shared, logits if gated else None, self.experts)
+        return self._combined(ctx, residual, y, weights, shared, logits if self.shared_gate_name is not None else None)
+
+    def _combined(self, ctx, residual, y, weights, shared, gate_logits):
+        """The stream with the weighted sum added; where its rows in the compute type are read next, the same launch leaves them."""
+        if not ctx.rows_wanted:
+            return ctx.ops.moe_combine(residual, y, weights, shared, gate_logits, self.experts)
+        x, rows = ctx.ops.moe_combine(residual, y, weights, shared, gate_logits, self.experts, rows_dtype=ctx.dtype)
+        ctx.note_rows(x, rows)
+        return x
 
     def branches(self, ctx, h):
         import torch

@@ -21,6 +21,9 @@ of its own, builds one of these for itself and calls `rotate`.
 """
 from __future__ import annotations
 
+import math
+from fractions import Fraction
+
 from .base import Position, WeightSpec, register_part
 
 
@@ -57,7 +60,6 @@ class Rotary(Position):
     def __init__(self, prefix: str = "", dims: int = 0, base: float = 10000.0, scaling: dict | None = None,
                  interleaved: bool = False):
         super().__init__(prefix)
-        import math
         self.dims, self.base, self.interleaved = int(dims), float(base), bool(interleaved)
         if self.dims <= 0 or self.dims % 2:
             raise ValueError(f"rotary {prefix!r}: {self.dims} rotated dimensions (an even number)")
@@ -101,6 +103,25 @@ class Rotary(Position):
 
     def apply_qk(self, ctx, qkv, n_heads: int, kv_heads: int, head_dim: int) -> None:
         self.rotate(ctx, qkv, qkv, n_heads + kv_heads, 0, head_dim, 0, head_dim, head_dim)
+
+
+def distance_buckets(rows: int, far: float) -> list:
+    """The bucket of every distance 0, 1, 2, ... up to the first that falls in the last of `rows` buckets (everything
+    beyond lies there too): with half = rows // 2, a distance n below half has a bucket of its own, and n from half on
+    falls in min(rows - 1, half + floor(ln(n / half) / ln(far / half) * (rows - half))) (the distance buckets of T5, for
+    one direction: Raffel et al., "Exploring the Limits of Transfer Learning with a Unified Text-to-Text Transformer").  The
+    floor is decided in whole numbers, so that a distance on a bucket's border falls where the equation puts it."""
+    half = rows // 2
+    if rows < 2 or not far > half:
+        raise ValueError(f"distances up to {far} in {rows} buckets: at least two buckets, and more distances than half of them")
+    span, out = rows - half, list(range(half))
+    ratio = Fraction(far) / half
+    for k in range(1, span):            # bucket half + k begins at the first n with (n / half)^span >= (far / half)^k
+        n = max(len(out), int(half * float(ratio) ** (k / span)) - 2)
+        while Fraction(n, half) ** span < ratio ** k:
+            n += 1
+        out += [half + k - 1] * (n - len(out))
+    return out + [rows - 1]
 
 
 register_part("position", "rotary", Rotary)

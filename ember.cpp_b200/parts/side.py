@@ -42,8 +42,10 @@ class TokenSideInput(StreamAddon):
         self.w_norm = runtime.vector(get(self.norm_name))
 
     def forward(self, ctx, x):
+        rows = ctx.rows_of(x)
+        ctx.note_rows(None, None)          # (the stream is added to in place: rows noted for it are no longer its own)
         return ctx.ops.side_input(x, ctx.plan, self.table, self.layer * self.dim, self.dim, self.w_gate, self.w_proj,
-                                  self.w_norm, self.eps)
+                                  self.w_norm, self.eps, rows=rows)
 
 
 register_part("addon", "token_side_input", TokenSideInput)

@@ -27,7 +27,7 @@ class CpuOps:
         x = x.float()
         mean = x.mean(-1, keepdim=True)
         var = ((x - mean) ** 2).mean(-1, keepdim=True)
-        return ((x - mean) * torch.rsqrt(var + eps) * w + b).to(out_dtype)
+        return ((x - mean) * torch.rsqrt(var + eps) * w + (0.0 if b is None else b)).to(out_dtype)
 
     def linear(self, a, w, bias, act=None, residual=None, out_dtype=None):
         y = a.float() @ w.float().t()
@@ -67,7 +67,8 @@ class CpuOps:
             cache.v[page, :, p % PAGE, :] = qkv[t, q_w + kv_w:q_w + kv_w + kv_heads * vd].view(kv_heads, vd).to(cache.v.dtype)
 
     def attention(self, qkv, cache, plan, n_heads, kv_heads, head_dim, scale, window, out_dtype, store=False,
-                  keep_first=0, value_dim=None, slopes=None, sinks=None, chunk=0, head_scales=None, head_scales_positive=True):
+                  keep_first=0, value_dim=None, slopes=None, sinks=None, chunk=0, head_scales=None, head_scales_positive=True,
+                  dist_bias=None):
         keep_first = keep_first or 0
         if store:
             self.kv_store(qkv, cache, plan, n_heads, kv_heads, head_dim, value_dim)
@@ -95,6 +96,8 @@ class CpuOps:
                 sc = (k[:, h // rep, :] @ q[h]) * scale * (1.0 if head_scales is None else float(head_scales[h]))
                 if slopes is not None:
                     sc = sc - slopes[h] * (p - pos).float()
+                if dist_bias is not None:
+                    sc = sc + dist_bias[h][(p - pos).clamp(max=dist_bias.shape[1] - 1)]
                 if sinks is not None:       # one more term of the denominator, without a value
                     pr = torch.softmax(torch.cat([sc, sinks[h:h + 1]]), 0)[:-1]
                 else:
@@ -202,8 +205,8 @@ class CpuOps:
             v = unit(v.view(-1, kv_heads, value_dim)).reshape(-1, kv_heads * value_dim)
         return torch.cat([q, k, v], 1).to(out_dtype)
 
-    def gate_mul(self, a, proj, z_col, gate="sigmoid"):
-        z = proj[:, z_col:z_col + a.shape[1]].float()
+    def gate_mul(self, a, proj, z_col, gate="sigmoid", span=1):
+        z = proj[:, z_col:z_col + a.shape[1] // span].float().repeat_interleave(span, 1)
         return (a.float() * (torch.sigmoid(z) if gate == "sigmoid" else z * torch.sigmoid(z))).to(a.dtype)
 
     # ------------------------------------------------------------------ norms after the sum, sums over depth
@@ -226,7 +229,7 @@ class CpuOps:
         return y, stream, stream.to(dtype)
 
     def qkv_prepare(self, proj, plan, cache, heads, kv_heads, head_dim, value_dim, out_dtype, store, v_col=None, norm=None,
-                    q_gain=None, k_gain=None, eps=0.0, rotary=None, unit_after=False):
+                    q_gain=None, k_gain=None, eps=0.0, rotary=None, unit_after=False, mix=None, queries=True):
         T, q_w, k_w = plan.T, heads * head_dim, kv_heads * head_dim
         unit = lambda t: t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps)  # noqa: E731
 
@@ -248,9 +251,12 @@ class CpuOps:
         out[:, :q_w] = heads_of(0, heads, q_gain)
         if store:
             v0 = q_w + k_w if v_col is None else v_col
-            rows = torch.cat([out[:, :q_w], heads_of(q_w, kv_heads, k_gain), proj[:, v0:v0 + kv_heads * value_dim].float()], 1)
+            v = proj[:, v0:v0 + kv_heads * value_dim].float()
+            if mix is not None:
+                v = (1.0 - mix[1]) * v + mix[1] * mix[0].float()
+            rows = torch.cat([out[:, :q_w], heads_of(q_w, kv_heads, k_gain), v], 1)
             self.kv_store(rows, cache, plan, heads, kv_heads, head_dim, value_dim)
-        return out.to(out_dtype)
+        return out.to(out_dtype) if queries else None
 
     def poly_norm(self, z, four, eps, out_dtype):
         z = z.float()
@@ -360,11 +366,12 @@ class CpuOps:
 
     def latent_rows(self, down, plan, q_rank, q_norm, kv_norm, kv_rank, rot_dim, eps, rotary, cache, out_dtype):
         c_q = self.rmsnorm(down[:, :q_rank], q_norm, eps, out_dtype)
+        interleaved = rotary.interleaved
         if cache is not None:
             c = self.rmsnorm(down[:, q_rank:q_rank + kv_rank], kv_norm, eps, torch.float32)
             k_r = torch.zeros(down.shape[0], rot_dim)
             self.rotate(down, k_r, plan.positions, 1, q_rank + kv_rank, rot_dim, 0, rot_dim, rot_dim, rotary.freqs,
-                        rotary.magnitude, rotary.dims)
+                        rotary.magnitude, rotary.dims, interleaved=interleaved)
             g = cache.group_index
             for t in range(plan.T):
                 s = int(plan.token_seq[t])
@@ -384,7 +391,7 @@ class CpuOps:
                 (a[:, a_col + h * a_head: a_col + h * a_head + k].float() @ w[h].float().t()).to(out.dtype)
         return out
 
-    def latent_attention(self, rows, cache, plan, heads, kv_rank, rot_dim, scale, out_dtype):
+    def latent_attention(self, rows, cache, plan, heads, kv_rank, rot_dim, scale, out_dtype, window=0):
         g = cache.group_index
         out = torch.zeros(plan.T, heads * kv_rank)
         q = rows.float().view(plan.T, heads, kv_rank + rot_dim)
@@ -392,7 +399,8 @@ class CpuOps:
             s = int(plan.token_seq[t])
             if int(plan.seq_slot[s]) < 0:
                 continue
-            pos = torch.arange(0, int(plan.positions[t]) + 1)
+            p = int(plan.positions[t])
+            pos = torch.arange(max(0, p - window + 1) if window > 0 else 0, p + 1)
             pages = plan.pages[g][s, pos // PAGE].long()
             assert (pages >= 0).all(), "a position is read whose page is not held"
             c = cache.k[pages, 0, pos % PAGE, :].float()
@@ -431,28 +439,36 @@ class CpuOps:
             return table[:T].long()
         return table[tokens[:T].long()].long()            # [T, top]: the expert of every (token, choice) pair
 
-    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale, softmax=False):
-        if softmax:
+    def moe_pick(self, logits, correction, experts, top, groups, keep_groups, route_scale, scores="sigmoid", group_top=2):
+        if scores == "softmax":
             picked, chosen = (logits[:, :experts].float() + correction).topk(top, dim=-1)
             return chosen.to(torch.int32), torch.softmax(picked, -1) * route_scale
-        s = torch.sigmoid(logits[:, :experts].float())
+        z = logits[:, :experts].float()
+        s = torch.softmax(z, -1) if scores == "softmax_all" else torch.sigmoid(z)
         choice = s + correction
         per = experts // groups
         if groups > 1:
             grouped = choice.view(-1, groups, per)
-            score = grouped.topk(min(2, per), dim=-1).values.sum(-1)
+            score = grouped.topk(min(group_top, per), dim=-1).values.sum(-1)
             kept = score.topk(keep_groups, dim=-1).indices
             allowed = torch.zeros_like(score, dtype=torch.bool).scatter_(1, kept, True)
             choice = torch.where(allowed.repeat_interleave(per, dim=1), choice, torch.full_like(choice, -float("inf")))
         chosen = choice.topk(top, dim=-1).indices
         w = s.gather(1, chosen)
+        if scores == "softmax_all":
+            return chosen.to(torch.int32), w * route_scale
         return chosen.to(torch.int32), w / (w.sum(-1, keepdim=True) + 1e-20) * route_scale
 
-    def moe_combine(self, x, y, weights, shared, logits, gate_col):
+    def moe_combine(self, x, y, weights, shared, logits, gate_col, rows_dtype=None):
         out = x + (y * weights[:, :, None]).sum(1)
         if shared is not None:
             out = out + (shared if logits is None else shared * torch.sigmoid(logits[:, gate_col:gate_col + 1].float()))
-        return out
+        return out if rows_dtype is None else (out, out.to(rows_dtype))
+
+    def moe_up(self, h, w_up, routing, out_dtype, act):
+        assert act == "relu2"
+        T, top = routing.shape
+        return torch.stack([torch.relu(w_up[routing[t, k]].float() @ h[t].float()) ** 2 for t in range(T) for k in range(top)]).to(out_dtype)
 
     def moe_gate_up(self, h, w_gate_up, routing, out_dtype, limit=0.0, alpha=1.0, shift=0.0):
         T, top = routing.shape
@@ -522,7 +538,7 @@ class CpuOps:
             state[slot] = S
         return out
 
-    def side_input(self, x, plan, table, col, dim, w_gate, w_proj, w_norm, eps):
+    def side_input(self, x, plan, table, col, dim, w_gate, w_proj, w_norm, eps, rows=None):
         e = table[plan.tokens[:x.shape[0]].long(), col:col + dim].float()
         z = x.float() @ w_gate.float().t()
         g = 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3))) * e

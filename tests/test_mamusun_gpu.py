@@ -452,7 +452,7 @@ def test_the_routers_choice_weighs_by_a_softmax_over_the_chosen(ops, experts, to
     T = 300
     logits, bias = rnd(1, T, experts + 3, scale=2.0), rnd(2, experts, scale=1.5)      # columns behind the router's own are not read
     logits[0, :experts] = 500.0 + torch.arange(experts)                              # large logits: the softmax must not overflow
-    chosen, weights = ops.moe_pick(logits.cuda(), bias.cuda(), experts, top, 1, 1, 1.0, softmax=True)
+    chosen, weights = ops.moe_pick(logits.cuda(), bias.cuda(), experts, top, 1, 1, 1.0, scores="softmax")
     want_e, want_w = P.route(f64(logits[:, :experts] + bias), top)
     assert np.array_equal(chosen.cpu().numpy(), want_e)
     close(weights, want_w, 1e-5)
