@@ -254,6 +254,33 @@ MAMUSUN_SIZES = {
 }
 
 
+PODENEX_SIZES = {
+    # taps of the convolutions, buckets of distances; groups of experts / kept; values a layer of the per-layer token input
+    # (the attention over cached rows is MUZOZEN_SIZES')
+    "small": dict(conv=4, rows=32, groups=4, keep=2, side=64),
+    "medium": dict(conv=4, rows=32, groups=4, keep=2, side=128),
+}
+
+
+def podenex_config(size: str):
+    """A Podenex of the width, layer count, attention heads, chunk and window, experts and vocabulary of `DESIGN_SIZES[size]` and
+    the cached rows of `MUZOZEN_SIZES[size]`: a windowed attention with a sink, an attention over cached rows in a window, an
+    attention inside chunks with convolutions and a bias by distance, in turn, every one with routed experts and a shared one."""
+    z, m, r = DESIGN_SIZES[size], PODENEX_SIZES[size], MUZOZEN_SIZES[size]
+    heads = {"dim": z["dim"], "vdim": z["dim"], "heads": z["heads"], "kv_heads": z["kv_heads"], "scale": z["dim"] ** -0.5,
+             "mask": {"size": z["window"]}, "v_mix": True}
+    latent = {"heads": r["heads"], "dim": r["dim"], "rot_dim": r["rot"], "vdim": r["vdim"], "q_rank": r["q_rank"],
+              "kv_rank": r["kv_rank"], "scale": (r["dim"] + r["rot"]) ** -0.5, "rot": {"dims": r["rot"], "base": 500000.0},
+              "mask": {"size": z["window"]}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "shared": {"ff": z["shared_ff"]},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": m["groups"], "keep": m["keep"]}}}
+    kinds = (("attention_2", heads), ("latent_attention", latent),
+             ("attention", {**heads, "conv": m["conv"], "bias_max": z["window"] // 2, "bias_rows": m["rows"]}))
+    layers = [{"type": kinds[i % 3][0], "mixer": dict(kinds[i % 3][1]), "mlp": dict(moe)} for i in range(z["layers"])]
+    return {"architecture": "Podenex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "token_side": {"dim": m["side"]},
+            "layers": layers}
+
+
 def mamusun_config(size: str):
     """A Mamusun of the width, layer count, attention heads, window, inner sizes, experts and vocabulary of
     `DESIGN_SIZES[size]`: attention beside the recurrence with experts, an attention over all keys whose values are its keys
@@ -353,6 +380,8 @@ def design_configs(size: str, design: str = "nipolorn"):
         return (mamusun_config(size),) + design_configs(size)
     if design == "vipolix":
         return (vipolix_config(size),) + design_configs(size)
+    if design == "podenex":       # (Vipolix has the like attention, experts and token input, Muzozen the like cached rows)
+        return (podenex_config(size), vipolix_config(size), muzozen_config(size))
     z = DESIGN_SIZES[size]
     left = {"dim": z["dim"], "vdim": z["dim"], "heads": z["heads"], "kv_heads": z["kv_heads"], "scale": z["dim"] ** -0.5,
             "mask": {"size": z["window"], "keep_first": z["keep"]}}
@@ -486,7 +515,7 @@ def main() -> int:
                     help="time one bfloat16 product on every kernel that takes it, instead of the benchmark")
     ap.add_argument("--act", default=None, choices=[None, "gelu_tanh", "gelu_erf"], help="with --linear: the epilogue's activation")
     ap.add_argument("--residual", action="store_true", help="with --linear: add a float32 residual (the output is float32 then)")
-    ap.add_argument("--design", default=None, choices=["nipolorn", "muzozen", "sosutar", "vipolix", "mamusun"],
+    ap.add_argument("--design", default=None, choices=["nipolorn", "muzozen", "sosutar", "vipolix", "mamusun", "podenex"],
                     help="instead of the benchmark: prefill and decode throughput of this design beside a GPT-2 of equal size "
                          "(muzozen: beside a Nipolorn and a GPT-2 of equal size)")
     ap.add_argument("--design-size", default="medium", choices=sorted(DESIGN_SIZES), help="with --design: the layers' sizes")
