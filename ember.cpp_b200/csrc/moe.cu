@@ -17,10 +17,9 @@
 namespace {
 
 // ---------------------------------------------------------------------------- routing
-__global__ void __launch_bounds__(1024)
-moe_route_kernel(const int* __restrict__ tokens, const int* __restrict__ table, int n_pairs, int top, int experts,
-                 int vocab, int* __restrict__ pair_expert, int* __restrict__ offsets, int* __restrict__ sorted) {
-  extern __shared__ int sm_i[];  // count[experts], cursor[experts]
+// sm_i: count[experts], cursor[experts].  `table` may have been written by this block before its last barrier.
+__device__ __forceinline__ void route_pairs(int* sm_i, const int* __restrict__ tokens, const int* table, int n_pairs, int top, int experts,
+                                            int vocab, int* pair_expert, int* __restrict__ offsets, int* __restrict__ sorted) {
   int* count = sm_i;
   int* cursor = sm_i + experts;
   for (int e = threadIdx.x; e < experts; e += blockDim.x) count[e] = 0;
@@ -45,6 +44,13 @@ moe_route_kernel(const int* __restrict__ tokens, const int* __restrict__ table, 
   }
   __syncthreads();
   for (int q = threadIdx.x; q < n_pairs; q += blockDim.x) sorted[atomicAdd(&cursor[pair_expert[q]], 1)] = q;
+}
+
+__global__ void __launch_bounds__(1024)
+moe_route_kernel(const int* __restrict__ tokens, const int* __restrict__ table, int n_pairs, int top, int experts,
+                 int vocab, int* __restrict__ pair_expert, int* __restrict__ offsets, int* __restrict__ sorted) {
+  extern __shared__ int sm_i[];
+  route_pairs(sm_i, tokens, table, n_pairs, top, experts, vocab, pair_expert, offsets, sorted);
 }
 
 // ---------------------------------------------------------------------------- streaming form
@@ -352,14 +358,10 @@ __device__ __forceinline__ void warp_argmax(float& best, int& at) {
 
 enum : int { kScoresSigmoid = 0, kScoresChosen = 1, kScoresAll = 2 };
 
-__global__ void __launch_bounds__(32 * kPickWarps)
-moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int T, int experts, int top,
-                int groups, int keep, int group_top, float scale, int scores, int* __restrict__ chosen, float* __restrict__ weights) {
-  extern __shared__ float pick_sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x * kPickWarps + warp;
-  if (t >= T) return;
-  float* sc = pick_sm + (size_t)warp * (2 * experts + groups);
+// One warp, token t; sc: 2 * experts + groups floats of the warp's own.
+__device__ __forceinline__ void pick_token(float* sc, int t, int lane, const float* __restrict__ logits, int ld,
+                                           const float* __restrict__ correction, int experts, int top, int groups, int keep,
+                                           int group_top, float scale, int scores, int* chosen, float* weights) {
   float* ch = sc + experts;
   float* gs = ch + experts;
   const bool softmax = scores == kScoresChosen;
@@ -439,6 +441,31 @@ moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restric
   for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= f;
 }
 
+__global__ void __launch_bounds__(32 * kPickWarps)
+moe_pick_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int T, int experts, int top,
+                int groups, int keep, int group_top, float scale, int scores, int* __restrict__ chosen, float* __restrict__ weights) {
+  extern __shared__ float pick_sm[];
+  const int warp = threadIdx.x >> 5, t = blockIdx.x * kPickWarps + warp;
+  if (t >= T) return;
+  pick_token(pick_sm + (size_t)warp * (2 * experts + groups), t, threadIdx.x & 31, logits, ld, correction, experts, top, groups, keep,
+             group_top, scale, scores, chosen, weights);
+}
+
+// A step of few tokens: the choice and the pairs by expert in one launch of one block, `warps` of whose warps pick.
+__global__ void __launch_bounds__(1024)
+moe_pick_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int T, int experts, int top,
+                      int groups, int keep, int group_top, float scale, int scores, int warps, int* chosen, float* weights,
+                      int* pair_expert, int* offsets, int* sorted) {
+  extern __shared__ float pick_sm[];
+  const int warp = threadIdx.x >> 5;
+  if (warp < warps)
+    for (int t = warp; t < T; t += warps)
+      pick_token(pick_sm + (size_t)warp * (2 * experts + groups), t, threadIdx.x & 31, logits, ld, correction, experts, top, groups,
+                 keep, group_top, scale, scores, chosen, weights);
+  __syncthreads();
+  route_pairs(reinterpret_cast<int*>(pick_sm), nullptr, chosen, T * top, top, experts, T, pair_expert, offsets, sorted);
+}
+
 // rows (or null): out once more, in bfloat16.
 // grid (T): out = x + sum_k weights[t, k] y[t, k, :] (k ascending) + sigmoid(gate) * shared[t, :]
 __global__ void __launch_bounds__(256)
@@ -476,6 +503,29 @@ EMBER_API int ember_moe_pick(const float* logits, int ld, const float* correctio
   const cudaError_t e = launch_plain(moe_pick_kernel, dim3((T + kPickWarps - 1) / kPickWarps), dim3(32 * kPickWarps), smem, stream,
                                      logits, ld, correction, T, experts, top, groups, keep, group_top, scale, scores, chosen, weights);
   if (e != cudaSuccess) return ember_fail("moe_pick: %s", cudaGetErrorString(e));
+  return 0;
+}
+
+// The two in one launch, for few tokens; returns 2, having launched nothing, where they are many or the experts' scores do
+// not fit the block's shared memory (the caller then makes the two launches).
+EMBER_API int ember_moe_pick_route(const float* logits, int ld, const float* correction, int T, int experts, int top, int groups,
+                                   int keep, int group_top, float scale, int scores, int* chosen, float* weights, int* pair_expert,
+                                   int* offsets, int* sorted, cudaStream_t stream) {
+  EMBER_CHECK(scores >= 0 && scores <= 2 && (group_top == 1 || group_top == 2), "moe_pick: scores %d, group_top %d", scores, group_top);
+  EMBER_CHECK(scores != kScoresChosen || groups == 1, "moe_pick: a softmax over the chosen with %d groups", groups);
+  EMBER_CHECK(T > 0 && experts > 0 && experts <= 1024 && top >= 1 && top <= experts && ld >= experts,
+              "moe_pick: %d tokens, top %d of %d experts (at most 1024)", T, top, experts);
+  EMBER_CHECK(groups >= 1 && experts % groups == 0 && keep >= 1 && keep <= groups && (long long)keep * (experts / groups) >= top,
+              "moe_pick: %d groups of which %d are kept do not hold %d choices", groups, keep, top);
+  constexpr int kFew = 64, kRoom = 40 * 1024;
+  const int a_warp = (2 * experts + groups) * (int)sizeof(float);
+  const int warps = min(min(T, 32), kRoom / a_warp);
+  if (T > kFew || warps < min(T, 8)) return 2;
+  const size_t smem = (size_t)max(warps * a_warp, 2 * experts * (int)sizeof(int));
+  const int threads = max(32 * warps, 128);
+  const cudaError_t e = launch_plain(moe_pick_route_kernel, dim3(1), dim3(threads), smem, stream, logits, ld, correction, T, experts, top,
+                                     groups, keep, group_top, scale, scores, warps, chosen, weights, pair_expert, offsets, sorted);
+  if (e != cudaSuccess) return ember_fail("moe_pick_route: %s", cudaGetErrorString(e));
   return 0;
 }
 

@@ -36,6 +36,8 @@ _SIGNATURES = {
                                      _c_int, _c_void],
     "ember_moe_pick": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void, _c_void,
                        _c_void],
+    "ember_moe_pick_route": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void, _c_void,
+                             _c_void, _c_void, _c_void, _c_void],
     "ember_moe_up": [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                      _c_int, _c_void],
     "ember_post_norm": [_c_void, _c_float, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_float, _c_float,
@@ -1351,6 +1353,24 @@ class CudaOps:
                    int(top), int(groups), int(keep_groups), int(group_top), float(route_scale), self._SCORES[scores], chosen.data_ptr(),
                    weights.data_ptr())
         return chosen, weights
+
+    def moe_pick_route(self, logits, correction, experts, top, groups, keep_groups, route_scale, scores="sigmoid", group_top=2):
+        """`moe_pick` and `moe_route` of its choice: (weights, routing); one launch for few tokens."""
+        T = logits.shape[0]
+        if T <= 64 and logits.dtype == torch.float32 and correction.dtype == torch.float32 and correction.numel() == experts:
+            pairs = T * top
+            buf = torch.empty(3 * pairs + experts + 1, dtype=torch.int32, device=logits.device)
+            chosen, pair_expert, order = buf[:pairs], buf[pairs:2 * pairs], buf[2 * pairs:3 * pairs]
+            offsets = buf[3 * pairs:]
+            weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
+            rc = self._call("ember_moe_pick_route", self._dense(logits, "logits").data_ptr(), logits.shape[1], correction.data_ptr(), T,
+                            int(experts), int(top), int(groups), int(keep_groups), int(group_top), float(route_scale),
+                            self._SCORES[scores], chosen.data_ptr(), weights.data_ptr(), pair_expert.data_ptr(), offsets.data_ptr(),
+                            order.data_ptr(), allow=(2,))
+            if rc == 0:
+                return weights, (pair_expert, offsets, order, T, top, experts)
+        chosen, weights = self.moe_pick(logits, correction, experts, top, groups, keep_groups, route_scale, scores, group_top)
+        return weights, self.moe_route(None, T, chosen, experts, top)
 
     def moe_combine(self, x, y, weights, shared, logits, gate_col, rows_dtype=None):
         """x + sum_k weights[:, k] * y[:, k, :] (+ shared, times sigmoid(logits[:, gate_col]) where logits are given),

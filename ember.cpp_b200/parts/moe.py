@@ -181,9 +181,8 @@ class RoutedExperts(FeedForward):
 
     def _chosen(self, ctx, h, logits):
         ops = ctx.ops
-        chosen, weights = ops.moe_pick(logits, self.correction, self.experts, self.top, self.groups, self.keep_groups,
-                                       self.route_scale, scores=self.scores, group_top=self.group_top)
-        routing = ops.moe_route(None, ctx.plan.T, chosen, self.experts, self.top)
+        weights, routing = ops.moe_pick_route(logits, self.correction, self.experts, self.top, self.groups, self.keep_groups,
+                                              self.route_scale, scores=self.scores, group_top=self.group_top)
         if self.gated:
             inner = ops.moe_gate_up(h, self.w_gate_up, routing, out_dtype=ctx.dtype, limit=self.limit, alpha=self.alpha,
                                     shift=self.shift)                                 # [T * top, inner]

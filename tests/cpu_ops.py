@@ -459,6 +459,10 @@ class CpuOps:
             return chosen.to(torch.int32), w * route_scale
         return chosen.to(torch.int32), w / (w.sum(-1, keepdim=True) + 1e-20) * route_scale
 
+    def moe_pick_route(self, logits, correction, experts, top, groups, keep_groups, route_scale, scores="sigmoid", group_top=2):
+        chosen, weights = self.moe_pick(logits, correction, experts, top, groups, keep_groups, route_scale, scores, group_top)
+        return weights, self.moe_route(None, logits.shape[0], chosen, experts, top)
+
     def moe_combine(self, x, y, weights, shared, logits, gate_col, rows_dtype=None):
         out = x + (y * weights[:, :, None]).sum(1)
         if shared is not None:

@@ -358,6 +358,21 @@ def test_the_routers_choice_by_a_softmax_over_all(ops, experts, top, groups, kee
     close(weights, want_w, 1e-5)
 
 
+@pytest.mark.parametrize("scores, groups, keep, group_top", [("softmax_all", 4, 2, 1), ("sigmoid", 8, 3, 2), ("softmax", 1, 1, 2)])
+@pytest.mark.parametrize("T, experts, top", [(1, 8, 2), (8, 32, 2), (64, 16, 6), (33, 160, 6), (5, 1024, 8)])
+def test_choice_and_sort_in_one_launch_equal_the_two(ops, scores, groups, keep, group_top, T, experts, top):
+    logits, corr = rnd(1, T, experts + 3, scale=2.0).cuda(), rnd(2, experts, scale=0.1).cuda()
+    args = (corr, experts, top, groups, keep, 1.5, scores, group_top)
+    if top > keep * (experts // groups):
+        pytest.skip("the kept groups hold fewer experts")
+    chosen, want = ops.moe_pick(logits, *args)
+    weights, (pair_expert, offsets, order, *_) = ops.moe_pick_route(logits, *args)
+    assert torch.equal(weights, want) and torch.equal(pair_expert.view(T, top), chosen)
+    counts = torch.bincount(chosen.view(-1).long(), minlength=experts).cumsum(0)
+    assert offsets[0] == 0 and torch.equal(offsets[1:].long(), counts) and sorted(order.tolist()) == list(range(T * top))
+    assert torch.equal(chosen.view(-1)[order.long()], chosen.view(-1).sort().values)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T, width, inner, experts, top", [(3, 64, 24, 6, 3), (70, 64, 24, 6, 3), (200, 96, 130, 4, 2), (40, 60, 14, 5, 2)])
 def test_experts_without_a_gate_and_their_weighted_sum(ops, dtype, T, width, inner, experts, top):
